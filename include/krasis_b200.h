@@ -361,6 +361,10 @@ KB2_API int kb2_mla_forward(kb2_mla* h, int layer, const void* hidden_dev, const
 KB2_API int kb2_fmha_latent(const void* q_dev, const void* kv_up_dev, const void* kpe_dev, void* out_dev, int32_t M, int32_t q_start,
                             int32_t kv_len, int32_t num_heads, float sm_scale, int32_t window, const float* sinks_dev, int32_t device,
                             void* stream);
+/* The same with a gate per head: out[i, h, :] is multiplied by sigmoid(gate_dev[i * gate_ld + h]) (fp32; NULL: no gate). */
+KB2_API int kb2_fmha_latent_gated(const void* q_dev, const void* kv_up_dev, const void* kpe_dev, void* out_dev, int32_t M, int32_t q_start,
+                                  int32_t kv_len, int32_t num_heads, float sm_scale, int32_t window, const float* sinks_dev,
+                                  const float* gate_dev, int64_t gate_ld, int32_t device, void* stream);
 
 /* Attention core on dense BF16 rows for heads that carry several attention maps (keys per map, shared values): q [M][num_q * 128] with
  * num_q = heads * maps query vectors laid out head by head, map by map; k [kv_len][num_kv_heads * maps * 128]; v [kv_len][num_kv_heads *
@@ -380,6 +384,13 @@ KB2_API int kb2_fmha_maps_softcap(const void* q_dev, const void* k_dev, const vo
 KB2_API int kb2_fmha_maps_sink(const void* q_dev, const void* k_dev, const void* v_dev, float* out_dev, int32_t M, int32_t q_start,
                                int32_t kv_len, int32_t num_q, int32_t num_kv_heads, int32_t maps, int32_t v_dim, float sm_scale,
                                float softcap, int32_t window, const float* sinks_dev, float* lse_dev, int32_t device, void* stream);
+
+/* The same with a penalty that grows with the distance: slopes_dev[v] * (position - key) is taken off query vector v's (capped) score
+ * (fp32 [num_q], may be null). */
+KB2_API int kb2_fmha_maps_slopes(const void* q_dev, const void* k_dev, const void* v_dev, float* out_dev, int32_t M, int32_t q_start,
+                                 int32_t kv_len, int32_t num_q, int32_t num_kv_heads, int32_t maps, int32_t v_dim, float sm_scale,
+                                 float softcap, int32_t window, const float* sinks_dev, float* lse_dev, const float* slopes_dev, int32_t device,
+                                 void* stream);
 
 /* GEMM -> reduce-scatter fused (head-parallel attention under token sharding): after kb2_{gdn,gqa,mla}_set_output_scatter the
  * block's out_proj GEMM stores every output row straight into the receive buffer of the rank that owns the token

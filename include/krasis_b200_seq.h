@@ -64,12 +64,13 @@ KB2SEQ_API int kb2_seq_latent_prep(float* proj, long long ldp, int T, int H, int
  * (sinks may be null: ordinary softmax).
  * With cu != NULL the tokens of sequences whose portion has skip_from tokens or more are left out (another kernel serves them).
  * nsplit > 1 cuts every token's key range into nsplit pieces that run as separate blocks (steps of few tokens: decoding) and are merged
- * by a second kernel; part_acc [T][nsplit][H][r] and part_ml [T][nsplit][H][2] (fp32) hold the pieces. */
+ * by a second kernel; part_acc [T][nsplit][H][r] and part_ml [T][nsplit][H][2] (fp32) hold the pieces.
+ * gate (may be null): out[t, h, :] is multiplied by sigmoid(gate[t * ldg + h]). */
 KB2SEQ_API int kb2_seq_latent_window_attn(const float* q_abs, const float* proj, long long ldp, int T, int H, int dn, int dr, int r,
                                           const void* ckv, const void* kr, int dt_cache, const int* positions, const int* seq_of,
                                           const int* pages, int max_pages, int page_size, const float* sinks, float scale, int window,
                                           float* out, const int* cu, int skip_from, int nsplit, float* part_acc, float* part_ml,
-                                          void* stream);
+                                          const float* gate, long long ldg, void* stream);
 
 /* out[t, c] = silu(causal conv over time of proj[:, c], K taps) for c < C; tail [slots][C][K - 1] is read, then advanced */
 KB2SEQ_API int kb2_seq_conv_silu(const float* proj, long long ldp, int T, int S, int C, int K, const float* taps, float* tail,
@@ -134,12 +135,13 @@ KB2SEQ_API int kb2_seq_kv_pool(const void* kc, const void* vc, void* kp, void* v
  * softcap > 0: a score s (after the scale) becomes softcap tanh(s / softcap).
  * sinks [H] (may be null): the softmax denominator of head h also holds exp(sinks[h]) (unscaled, no value).
  * pool > 0 (needs chunk == 0): beside the window's keys a token sees one key and value per block of `pool` positions that lies wholly
- * before its window (b pool + pool - 1 <= pos - window), read from the pooled pools kp / vp (see kb2_seq_kv_pool), in the same softmax. */
+ * before its window (b pool + pool - 1 <= pos - window), read from the pooled pools kp / vp (see kb2_seq_kv_pool), in the same softmax.
+ * slopes [H] (may be null; needs pool == 0): slopes[h] * (pos - j) is taken off head h's score of key j, after the cap. */
 KB2SEQ_API int kb2_seq_paged_attn(const float* proj, long long ldp, int T, int H, int G, int M, int d, int dv, const void* kc,
                                   const void* vc, int dt_cache, const int* positions, const int* seq_of, const int* pages, int max_pages,
                                   int page_size, float scale, int chunk, int window, float* out, int nsplit, float* part_acc,
                                   float* part_ml, const int* cu, int skip_from, float softcap, const float* sinks, int pool, const void* kp,
-                                  const void* vp, int pool_only, void* stream);
+                                  const void* vp, int pool_only, const float* slopes, void* stream);
 
 /* pool_only 1 (above; needs cu, nsplit 1 and the piece buffers): the pass that follows a tensor-core attention over the window of long
  * portions — only the tokens of sequences whose portion has skip_from tokens or more, only their pooled blocks, no sink; the result stays
@@ -162,12 +164,13 @@ KB2SEQ_API int kb2_seq_attn_finish(const float* a, const float* part_acc, const 
 KB2SEQ_API int kb2_seq_glu(const void* in, int dt_in, long long ld_in, void* out, int dt_out, long long rows, int F, int kind, float limit,
                            float alpha, const int* n_tiles, int tile_rows, void* stream);
 
-/* Router: z [T, ldz] fp32 logits of E outputs -> ids [T, top], weights [T, top].  score_kind 0 softmax, 1 sigmoid; choice = score +
+/* Router: z [T, ldz] fp32 logits of E outputs (bias [E], may be null, is added first) -> ids [T, top], weights [T, top].
+ * score_kind 0 softmax, 1 sigmoid, 2 the logit itself (weights are then the softmax over the chosen logits alone); choice = score +
  * correction (may be null); groups > 1: E / groups neighbours form a group, only the `keep` groups with the largest group score
  * (group_kind 0: the group's largest choice, 1: the sum of its two largest) can be chosen; weights are the chosen scores (without
  * correction), divided by their sum (+ 1e-20) if renorm, times out_scale. */
 KB2SEQ_API int kb2_seq_route(const float* z, long long ldz, int T, int E, const float* correction, int score_kind, int groups, int keep,
-                             int top, int renorm, float out_scale, int* ids, float* weights, int group_kind, void* stream);
+                             int top, int renorm, float out_scale, int* ids, float* weights, int group_kind, const float* bias, void* stream);
 
 /* Routed experts.  moe_bin: slots = T * top entries of ids; ids outside [0, E) are left out (identity experts).  Each expert's slots
  * form a run of rows padded to whole tiles of tile_rows (a multiple of kb2_seq_moe_tile_rows()): offs [E + 1], tile_expert [max_rows / tile], n_tiles [1],
@@ -229,6 +232,13 @@ KB2SEQ_API int kb2_seq_branch_merge(const float* a, const float* b, const float*
  * x <- sum_j coef[j] stack[j] (j < n, ascending), and h = x / rms(x) * w in dt_h if w is given. */
 KB2SEQ_API int kb2_seq_depth_mix(float* stack, long long stride, int n, const float* coef, float* x, const float* y, const float* w, void* h,
                                  int dt_h, int T, int W, float eps, void* stream);
+
+/* Residual stream of n copies, xs [T][n][W] fp32 (1 <= n <= 32).  x0 [T, W] given: every copy starts as x0 (xs is written, not read).
+ * y [T, W] given (with mix [n][n], indexed [from][to], and out [n]): copy t <- sum_s mix[s, t] copy_s + out[t] y, all copies from the old
+ * ones.  Then u = sum_s read[s] copy_s (read null: their plain sum); h = u / sqrt(mean(u^2) + eps) * (w_shift + w) in dt_h if w is given,
+ * h = u if it is not; h may be null. */
+KB2SEQ_API int kb2_seq_stream_mix(float* xs, int n, const float* x0, const float* y, const float* mix, const float* out, const float* read,
+                                  const float* w, float w_shift, void* h, int dt_h, int T, int W, float eps, void* stream);
 
 #ifdef __cplusplus
 }

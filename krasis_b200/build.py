@@ -5,8 +5,10 @@ Two targets, so that a model only compiles what it runs on:
   "seq"   libkrasis_b200_seq.so   ragged-batch sequence operators (csrc/seq_ops.cu, seq_mix.cu, seq_rec.cu): norms, generic GEMM, windowed
                                   latent attention with an optional sink, short convolution + gated delta rule (decay per head or per
                                   key channel) with state slots, per-head paged multi-map attention (score cap, sink, pooled blocks
-                                  before the window, rotated values), gated and ungated linear units, router and routed experts,
-                                  gated linear attention and selective scan with state slots, side-by-side mixers, depth average
+                                  before the window, rotated values, distance penalty), gated and ungated linear units, router and
+                                  routed experts,
+                                  gated linear attention and selective scan with state slots, side-by-side mixers, depth average,
+                                  several mixed copies of the residual stream
 nvcc cross-compiles without a GPU.  The .so files are git-ignored; a missing or stale one is rebuilt on demand.
 """
 import hashlib

@@ -46,9 +46,10 @@ cudaError_t launch_gqa_core(const GqaDims& g, const void* q_raw, const void* k_r
                             void* v_cache, void* k_bf, void* v_bf, void* attn_out, int M, int q_start, int kv_len,
                             cudaStream_t s);
 cudaError_t launch_fmha_latent(const void* q, const void* kv_up, const void* kpe, void* out, int M, int q_start, int kv_len, int nh,
-                               float sm_scale, int window, const float* sinks, cudaStream_t s);
+                               float sm_scale, int window, const float* sinks, cudaStream_t s, const float* head_gate = nullptr, long long ldg = 0);
 cudaError_t launch_fmha_maps(const void* q, const void* k, const void* v, float* out_f32, int M, int q_start, int kv_len, int nq, int nkv,
-                             int maps, int dv, float sm_scale, int window, cudaStream_t s, float softcap = 0.f, const float* sinks = nullptr, float* lse_out = nullptr);
+                             int maps, int dv, float sm_scale, int window, cudaStream_t s, float softcap = 0.f, const float* sinks = nullptr, float* lse_out = nullptr,
+                             const float* slopes = nullptr);
 struct MlaDims {
   int H, nh, nope, rope, dv, lora;
   float eps;
@@ -646,16 +647,23 @@ KB2_API int kb2_mla_forward(kb2_mla* h, int layer, const void* hidden_dev, const
   return KB2_OK;
 }
 
-KB2_API int kb2_fmha_latent(const void* q_dev, const void* kv_up_dev, const void* kpe_dev, void* out_dev, int32_t M, int32_t q_start,
-                            int32_t kv_len, int32_t num_heads, float sm_scale, int32_t window, const float* sinks_dev, int32_t device,
-                            void* stream) {
+KB2_API int kb2_fmha_latent_gated(const void* q_dev, const void* kv_up_dev, const void* kpe_dev, void* out_dev, int32_t M, int32_t q_start,
+                                  int32_t kv_len, int32_t num_heads, float sm_scale, int32_t window, const float* sinks_dev,
+                                  const float* gate_dev, int64_t gate_ld, int32_t device, void* stream) {
   if (!q_dev || !kv_up_dev || !kpe_dev || !out_dev) return failf(KB2_ERR_VALUE, "null argument");
   if (M <= 0 || num_heads <= 0 || q_start < 0 || kv_len != q_start + M || window <= 0)
     return failf(KB2_ERR_VALUE, "fmha_latent: need M > 0, kv_len == q_start + M, window > 0 (M=%d q_start=%d kv_len=%d)", M, q_start, kv_len);
   CUDA_TRY(cudaSetDevice(device));
   CUDA_TRY(launch_fmha_latent(q_dev, kv_up_dev, kpe_dev, out_dev, M, q_start, kv_len, num_heads, sm_scale, window, sinks_dev,
-                              (cudaStream_t)stream));
+                              (cudaStream_t)stream, gate_dev, gate_ld));
   return KB2_OK;
+}
+
+KB2_API int kb2_fmha_latent(const void* q_dev, const void* kv_up_dev, const void* kpe_dev, void* out_dev, int32_t M, int32_t q_start,
+                            int32_t kv_len, int32_t num_heads, float sm_scale, int32_t window, const float* sinks_dev, int32_t device,
+                            void* stream) {
+  return kb2_fmha_latent_gated(q_dev, kv_up_dev, kpe_dev, out_dev, M, q_start, kv_len, num_heads, sm_scale, window, sinks_dev, nullptr, 0, device,
+                               stream);
 }
 
 KB2_API int kb2_fmha_maps_softcap(const void* q_dev, const void* k_dev, const void* v_dev, float* out_dev, int32_t M, int32_t q_start,
@@ -672,9 +680,10 @@ KB2_API int kb2_fmha_maps_softcap(const void* q_dev, const void* k_dev, const vo
   return KB2_OK;
 }
 
-KB2_API int kb2_fmha_maps_sink(const void* q_dev, const void* k_dev, const void* v_dev, float* out_dev, int32_t M, int32_t q_start,
-                               int32_t kv_len, int32_t num_q, int32_t num_kv_heads, int32_t maps, int32_t v_dim, float sm_scale,
-                               float softcap, int32_t window, const float* sinks_dev, float* lse_dev, int32_t device, void* stream) {
+KB2_API int kb2_fmha_maps_slopes(const void* q_dev, const void* k_dev, const void* v_dev, float* out_dev, int32_t M, int32_t q_start,
+                                 int32_t kv_len, int32_t num_q, int32_t num_kv_heads, int32_t maps, int32_t v_dim, float sm_scale,
+                                 float softcap, int32_t window, const float* sinks_dev, float* lse_dev, const float* slopes_dev, int32_t device,
+                                 void* stream) {
   if (!q_dev || !k_dev || !v_dev || !out_dev) return failf(KB2_ERR_VALUE, "null argument");
   if (M <= 0 || num_q <= 0 || num_kv_heads <= 0 || maps <= 0 || num_q % maps || (num_q / maps) % num_kv_heads || q_start < 0 ||
       kv_len != q_start + M || window <= 0 || (v_dim != 128 && v_dim != 256) || !(softcap >= 0.f) || !(sm_scale > 0.f))
@@ -682,8 +691,15 @@ KB2_API int kb2_fmha_maps_sink(const void* q_dev, const void* k_dev, const void*
                  M, q_start, kv_len, v_dim);
   CUDA_TRY(cudaSetDevice(device));
   CUDA_TRY(launch_fmha_maps(q_dev, k_dev, v_dev, out_dev, M, q_start, kv_len, num_q, num_kv_heads, maps, v_dim, sm_scale, window,
-                            (cudaStream_t)stream, softcap, sinks_dev, lse_dev));
+                            (cudaStream_t)stream, softcap, sinks_dev, lse_dev, slopes_dev));
   return KB2_OK;
+}
+
+KB2_API int kb2_fmha_maps_sink(const void* q_dev, const void* k_dev, const void* v_dev, float* out_dev, int32_t M, int32_t q_start,
+                               int32_t kv_len, int32_t num_q, int32_t num_kv_heads, int32_t maps, int32_t v_dim, float sm_scale,
+                               float softcap, int32_t window, const float* sinks_dev, float* lse_dev, int32_t device, void* stream) {
+  return kb2_fmha_maps_slopes(q_dev, k_dev, v_dev, out_dev, M, q_start, kv_len, num_q, num_kv_heads, maps, v_dim, sm_scale, softcap, window,
+                              sinks_dev, lse_dev, nullptr, device, stream);
 }
 
 KB2_API int kb2_fmha_maps(const void* q_dev, const void* k_dev, const void* v_dev, float* out_dev, int32_t M, int32_t q_start,

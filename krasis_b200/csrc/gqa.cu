@@ -186,8 +186,11 @@ __global__ void __launch_bounds__(kFThreads, 1)
                     float* __restrict__ out_f32 = nullptr,       // if given, the output rows are written here in fp32 (no gate), not to `out`
                     float cap_in = 0.f, float cap_out = 0.f,     // soft cap: a raw score s becomes cap_out * tanh(s * cap_in) with
                                                                  // cap_in = sm_scale / cap, cap_out = cap / sm_scale (0: no cap)
-                    float* __restrict__ lse_out = nullptr) {     // if given, [M][nh]: log(sum of exp(scaled scores)) of every row (the sink
+                    float* __restrict__ lse_out = nullptr,       // if given, [M][nh]: log(sum of exp(scaled scores)) of every row (the sink
                                                                  // included), so that a caller can merge further keys into the softmax
+                    const float* __restrict__ slopes = nullptr,  // if given, [nh]: slopes[head] * (q_pos - key) is taken off the scaled score
+                    const float* __restrict__ head_gate = nullptr, long long ldg = 0) {   // if given, [M][ldg]: head h's output rows are
+                                                                 // multiplied by sigmoid(head_gate[row][h])
   using L = FmhaSmem<DQ, DV>;
   constexpr int D = DQ;
   constexpr int NC = DQ / 64;                      // 64-wide d chunks of q/k
@@ -357,6 +360,8 @@ __global__ void __launch_bounds__(kFThreads, 1)
     float* xchg = reinterpret_cast<float*>(smem + L::kOffXchg);
     constexpr int KH = kFK / 2, OH = DV / 2;
     float m_ref = -INFINITY, l_sum = 0.f;
+    // the penalty in units of the raw scores, so that the scale folded into the exponent applies to both
+    const float slope = slopes != nullptr ? slopes[head] * 1.4426950408889634f / sm_scale_log2 : 0.f;
     uint32_t sf_phase = 0;
     // PV completions observed so far on each of the two pv_done barriers.  P is double-buffered, so a tile only has to
     // wait for PV(it-2) (its P buffer is free again) — and for PV(it-1) in the rare case it rescales O.  A thread never
@@ -393,6 +398,11 @@ __global__ void __launch_bounds__(kFThreads, 1)
         for (int jj = 0; jj < KH; ++jj) s[jj] = cap_out * (1.f - __fdividef(2.f, ex2_approx(s[jj] * c2) + 1.f));
       }
       const int key0 = (it + tile0) * kFK + hf * KH;
+      if (slope != 0.f) {
+        const float back = (float)(key0 - q_pos);          // minus the distance; invisible keys are masked below whatever this gives
+#pragma unroll
+        for (int jj = 0; jj < KH; ++jj) s[jj] = fmaf(slope, back + (float)jj, s[jj]);
+      }
       // causal / length / window mask only where a key of this half-tile can be invisible to a row of this warp (warp-uniform)
       if (key0 + KH - 1 > q_start + q0 + q * 32 || key0 + KH > kv_len || key0 + window <= q_start + q0 + q * 32 + 31) {
 #pragma unroll
@@ -460,8 +470,9 @@ __global__ void __launch_bounds__(kFThreads, 1)
         lse_out[(long long)qi * g.nh + head] = l_sum > 0.f ? (m_ref + log2f(l_sum)) * 0.6931471805599453f : -INFINITY;
       if (n_tiles >= 2) pv_wait((n_tiles - 2) & 1, (uint32_t)((n_tiles - 2) / 2 + 1));
       pv_wait((n_tiles - 1) & 1, (uint32_t)((n_tiles - 1) / 2 + 1));
-      const float inv_l = l_sum > 0.f ? 1.0f / l_sum : 0.f;
       const bool live = qi < M;
+      float inv_l = l_sum > 0.f ? 1.0f / l_sum : 0.f;
+      if (head_gate != nullptr && live) inv_l *= 1.0f / (1.0f + expf(-head_gate[(long long)qi * ldg + head]));
       const long long obase = (long long)qi * g.nh * DV + (long long)head * DV;
       const long long gbase = (long long)qi * g.nh * D * 2 + (long long)head * 2 * D + D;   // gate half of q_raw
       const bool gated = g.gated != 0;
@@ -728,9 +739,10 @@ cudaError_t launch_mla_core(const MlaDims& m, void* q_full, const void* kv_a, co
 // The attention core alone on dense BF16 rows, for callers that keep their own cache: q [M][nh*192] (per head 128 unrotated + 64
 // rotated), kv_up [kv_len][nh*256] = [k_nope of every head | v of every head], kpe [kv_len][64] (the rotated key part all heads share),
 // out [M][nh*128].  Query i stands at position q_start + i of the kv rows and sees the keys with 0 <= position - key < window;
-// sinks (fp32 [nh], may be null) adds exp(sink) to each head's softmax denominator.
+// sinks (fp32 [nh], may be null) adds exp(sink) to each head's softmax denominator.  head_gate (fp32 [M][ldg], may be null): head h's
+// output row i is multiplied by sigmoid(head_gate[i][h]).
 cudaError_t launch_fmha_latent(const void* q, const void* kv_up, const void* kpe, void* out, int M, int q_start, int kv_len, int nh,
-                               float sm_scale, int window, const float* sinks, cudaStream_t s) {
+                               float sm_scale, int window, const float* sinks, cudaStream_t s, const float* head_gate, long long ldg) {
   if (M <= 0 || nh <= 0 || q_start < 0 || kv_len != q_start + M || window <= 0) return cudaErrorInvalidValue;
   static PerDeviceOnce once;
   if (const int dev = once.pending(); dev >= 0) {
@@ -750,7 +762,8 @@ cudaError_t launch_fmha_latent(const void* q, const void* kv_up, const void* kpe
   dim3 grid((M + kFQ - 1) / kFQ, nh);
   KernelSpan ks(K_FMHA, s);
   gqa_fmha_kernel<192, 128, true><<<grid, kFThreads, FmhaSmem<192, 128>::kTotal, s>>>(
-      tq, tk, tpe, tk, g, nullptr, (__nv_bfloat16*)out, M, q_start, kv_len, sm_scale * 1.4426950408889634f, 0, nh * 128, window, sinks);
+      tq, tk, tpe, tk, g, nullptr, (__nv_bfloat16*)out, M, q_start, kv_len, sm_scale * 1.4426950408889634f, 0, nh * 128, window, sinks, 1,
+      nullptr, 0.f, 0.f, nullptr, nullptr, head_gate, ldg);
   return cudaGetLastError();
 }
 
@@ -758,9 +771,11 @@ cudaError_t launch_fmha_latent(const void* q, const void* kv_up, const void* kpe
 // vectors (head by head, map by map), k [kv_len][nkv * maps * 128], v [kv_len][nkv * dv], dv 128 or 256; out_f32 [M][nq * dv] fp32.
 // Query i stands at position q_start + i of the kv rows and sees the keys with 0 <= position - key < window.
 // softcap > 0: a scaled score s becomes softcap * tanh(s / softcap).  sinks (fp32 [nq], may be null): exp(sink) joins each query vector's
-// softmax denominator.  lse_out (fp32 [M][nq], may be null): the logarithm of that denominator per row.
+// softmax denominator.  lse_out (fp32 [M][nq], may be null): the logarithm of that denominator per row.  slopes (fp32 [nq], may be null):
+// slopes[query vector] * (distance to the key) is taken off the (capped) score.
 cudaError_t launch_fmha_maps(const void* q, const void* k, const void* v, float* out_f32, int M, int q_start, int kv_len, int nq, int nkv,
-                             int maps, int dv, float sm_scale, int window, cudaStream_t s, float softcap, const float* sinks, float* lse_out) {
+                             int maps, int dv, float sm_scale, int window, cudaStream_t s, float softcap, const float* sinks, float* lse_out,
+                             const float* slopes) {
   if (!(softcap >= 0.f) || !(sm_scale > 0.f)) return cudaErrorInvalidValue;
   const float cap_in = softcap > 0.f ? sm_scale / softcap : 0.f, cap_out = softcap > 0.f ? softcap / sm_scale : 0.f;
   if (M <= 0 || nq <= 0 || nkv <= 0 || maps <= 0 || nq % maps || (nq / maps) % nkv || q_start < 0 || kv_len != q_start + M || window <= 0 ||
@@ -787,10 +802,10 @@ cudaError_t launch_fmha_maps(const void* q, const void* k, const void* v, float*
   const float sl2 = sm_scale * 1.4426950408889634f;
   if (dv == 256)
     gqa_fmha_kernel<128, 256, false><<<grid, kFThreads, FmhaSmem<128, 256>::kTotal, s>>>(tq, tk, tk, tv, g, nullptr, nullptr, M, q_start, kv_len,
-                                                                                          sl2, 0, 0, window, sinks, maps, out_f32, cap_in, cap_out, lse_out);
+                                                                                          sl2, 0, 0, window, sinks, maps, out_f32, cap_in, cap_out, lse_out, slopes);
   else
     gqa_fmha_kernel<128, 128, false><<<grid, kFThreads, FmhaSmem<128, 128>::kTotal, s>>>(tq, tk, tk, tv, g, nullptr, nullptr, M, q_start, kv_len,
-                                                                                          sl2, 0, 0, window, sinks, maps, out_f32, cap_in, cap_out, lse_out);
+                                                                                          sl2, 0, 0, window, sinks, maps, out_f32, cap_in, cap_out, lse_out, slopes);
   return cudaGetLastError();
 }
 

@@ -9,16 +9,17 @@
 //                          into pooled pools that share the page numbering
 //   paged_attn             softmax attention of every (head, map) query vector over the cached keys of its key/value head; the maps of
 //                          a head have keys of their own and share the values; keys j <= i of the same chunk and inside the window;
-//                          optional tanh cap on the scaled scores; optional sink per head in the denominator; optionally one pooled
-//                          key / value per block that lies wholly before the window, in the same softmax;
+//                          optional tanh cap on the scaled scores; optional penalty slope * distance per head; optional sink per head
+//                          in the denominator; optionally one pooled key / value per block that lies wholly before the window, in the
+//                          same softmax;
 //                          for steps of few tokens the key range is cut into pieces that run as separate blocks
 //   pool_merge             joins the pooled blocks' piece to a tensor-core result over the window by the two log-sum-exps
 //   attn_finish            merges the pieces, combines the maps with per-map coefficients (differential attention: 1, -lambda),
 //                          unit RMS norm per head, turning rotated values back by the query's position, output gate sigmoid(g) per
 //                          head or per element
 //   glu                    act(gate) * up in three flavours (tanh-GELU, SiLU, clamped swish with up + 1), or relu^2 without an up half
-//   route_topk             scores (softmax or sigmoid) -> + correction -> best groups (by their best or two best members) -> top-k
-//                          -> weights
+//   route_topk             logits (+ bias) -> scores (softmax, sigmoid, or the logits themselves) -> + correction -> best groups (by their
+//                          best or two best members) -> top-k -> weights (the scores, or a softmax over the chosen logits alone)
 //   moe_bin / moe_gemm / moe_gemv / moe_combine
 //                          tokens binned per expert in tiles of 64 rows, tile GEMMs that pick their expert's weights, a GEMV form for
 //                          steps of few tokens, and the weighted sum over a token's experts (identity experts return the input)
@@ -171,7 +172,8 @@ __global__ void __launch_bounds__(kPAThreads) paged_attn_kernel(
     const void* __restrict__ vc, int dt_cache, const int* __restrict__ positions, const int* __restrict__ seq_of,
     const int* __restrict__ pages, int max_pages, int page_size, float scale, int chunk, int window, float* __restrict__ out, int nsplit,
     float* __restrict__ part_acc, float* __restrict__ part_ml, const int* __restrict__ cu, int skip_from, float softcap,
-    const float* __restrict__ sinks, int pool, int rows_per_page, const void* __restrict__ kp, const void* __restrict__ vp, int pool_only) {
+    const float* __restrict__ sinks, int pool, int rows_per_page, const void* __restrict__ kp, const void* __restrict__ vp, int pool_only,
+    const float* __restrict__ slopes) {
   extern __shared__ __align__(16) float sm[];
   constexpr int KT = kPAKT;
   const long long t = blockIdx.x;
@@ -271,6 +273,8 @@ __global__ void __launch_bounds__(kPAThreads) paged_attn_kernel(
         for (int dd = 0; dd < d; ++dd) dot = fmaf(qh[dd], kk[dd], dot);
         sc = dot * scale;
         if (softcap > 0.f) sc = softcap * tanhf(sc / softcap);
+        // no pooled blocks beside slopes (checked by the host): entry j0 + lane of the key list is position j_lo + j0 + lane
+        if (slopes != nullptr) sc = fmaf(-slopes[g * (H / G) + (r0 + r) / M], (float)(pos - (j_lo + j0 + lane)), sc);
       }
       const float m_old = m_run[r];
       const float m_new = fmaxf(m_old, warp_max(sc));
@@ -483,14 +487,15 @@ __global__ void glu_bf16x8_kernel(const bf16* __restrict__ in, long long ld_in, 
 }
 
 // ------------------------------------------------------------------------------------------------ router
-// A warp per token.  s = softmax(z) (score_kind 0) or sigmoid(z) (1) over the E router outputs; choice c = s + correction; with
+// A warp per token.  z is the router product plus bias (bias may be null).  s = softmax(z) (score_kind 0), sigmoid(z) (1) or z itself (2)
+// over the E router outputs; choice c = s + correction; with
 // groups > 1 only the experts of the `keep` groups with the largest group score (their largest choice, or the sum of their two largest)
 // stay in play; the `top` largest choices are taken (ties: lower index); weights are the chosen s, divided by their sum (+ 1e-20) if
-// renorm, times out_scale.
+// renorm, times out_scale.  score_kind 2: the weights are the softmax over the chosen logits alone, times out_scale.
 __global__ void __launch_bounds__(128) route_topk_kernel(const float* __restrict__ z, long long ldz, int T, int E,
                                                          const float* __restrict__ correction, int score_kind, int groups, int keep,
                                                          int top, int renorm, float out_scale, int* __restrict__ ids,
-                                                         float* __restrict__ weights, int group_kind) {
+                                                         float* __restrict__ weights, int group_kind, const float* __restrict__ bias) {
   extern __shared__ float rsm[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
   const long long t = (long long)blockIdx.x * nw + warp;
@@ -501,18 +506,20 @@ __global__ void __launch_bounds__(128) route_topk_kernel(const float* __restrict
   const float* zr = z + t * ldz;
   if (score_kind == 0) {
     float mx = -INFINITY;
-    for (int e = lane; e < E; e += 32) mx = fmaxf(mx, zr[e]);
+    for (int e = lane; e < E; e += 32) mx = fmaxf(mx, zr[e] + (bias ? bias[e] : 0.f));
     mx = warp_max(mx);
     float sum = 0.f;
     for (int e = lane; e < E; e += 32) {
-      const float v = expf(zr[e] - mx);
+      const float v = expf(zr[e] + (bias ? bias[e] : 0.f) - mx);
       s[e] = v;
       sum += v;
     }
     sum = warp_sum(sum);
     for (int e = lane; e < E; e += 32) s[e] = s[e] / sum;
+  } else if (score_kind == 1) {
+    for (int e = lane; e < E; e += 32) s[e] = 1.f / (1.f + expf(-(zr[e] + (bias ? bias[e] : 0.f))));
   } else {
-    for (int e = lane; e < E; e += 32) s[e] = 1.f / (1.f + expf(-zr[e]));
+    for (int e = lane; e < E; e += 32) s[e] = zr[e] + (bias ? bias[e] : 0.f);
   }
   for (int e = lane; e < E; e += 32) c[e] = s[e] + (correction ? correction[e] : 0.f);
   __syncwarp();
@@ -548,7 +555,7 @@ __global__ void __launch_bounds__(128) route_topk_kernel(const float* __restrict
       if (gsc[e / gs] != INFINITY) c[e] = -INFINITY;
     __syncwarp();
   }
-  float wsum = 0.f;
+  float wsum = 0.f, z_top = 0.f;            // z_top: the largest chosen logit (score_kind 2)
   for (int it = 0; it < top; ++it) {
     float bv = -INFINITY;
     int bi = 0x7fffffff;
@@ -563,16 +570,21 @@ __global__ void __launch_bounds__(128) route_topk_kernel(const float* __restrict
       if (ov > bv || (ov == bv && oi < bi)) { bv = ov; bi = oi; }
     }
     const bool found = bi < E;
+    float wt = found ? s[bi] : 0.f;
+    if (score_kind == 2 && found) {         // exp of the distance to the first chosen logit; the sum below makes it a softmax
+      if (it == 0) z_top = wt;
+      wt = expf(wt - z_top);
+    }
     if (lane == 0) {
       ids[t * top + it] = found ? bi : -1;
-      weights[t * top + it] = found ? s[bi] : 0.f;
+      weights[t * top + it] = wt;
       if (found) c[bi] = -INFINITY;
     }
-    if (found) wsum += s[bi];
+    wsum += wt;
     __syncwarp();
   }
   if (lane == 0) {
-    const float f = (renorm ? 1.f / (wsum + 1e-20f) : 1.f) * out_scale;
+    const float f = (score_kind == 2 ? 1.f / wsum : renorm ? 1.f / (wsum + 1e-20f) : 1.f) * out_scale;
     if (f != 1.f)
       for (int it = 0; it < top; ++it) weights[t * top + it] *= f;
   }
@@ -798,7 +810,8 @@ KB2SEQ_API int kb2_seq_paged_attn(const float* proj, long long ldp, int T, int H
                                   const void* vc, int dt_cache, const int* positions, const int* seq_of, const int* pages, int max_pages,
                                   int page_size, float scale, int chunk, int window, float* out, int nsplit, float* part_acc,
                                   float* part_ml, const int* cu, int skip_from, float softcap, const float* sinks, int pool, const void* kp,
-                                  const void* vp, int pool_only, void* stream) {
+                                  const void* vp, int pool_only, const float* slopes, void* stream) {
+  if (slopes && pool > 0) return failf(KB2SEQ_ERR_VALUE, "paged_attn: a distance penalty and pooled blocks exclude each other");
   if (pool < 0 || (pool > 0 && (!kp || !vp || chunk > 0))) return failf(KB2SEQ_ERR_VALUE, "paged_attn: pooled blocks need their pools and no chunks");
   if (pool_only && (pool <= 0 || nsplit != 1 || !part_acc || !part_ml || !cu))
     return failf(KB2SEQ_ERR_VALUE, "paged_attn: the pass over the pooled blocks alone needs pool > 0, one key piece, the piece buffers and cu");
@@ -820,7 +833,7 @@ KB2SEQ_API int kb2_seq_paged_attn(const float* proj, long long ldp, int T, int H
   if ((long long)G * nrb > 65535) return failf(KB2SEQ_ERR_VALUE, "paged_attn: too many heads");
   paged_attn_kernel<<<dim3(T, G * nrb, nsplit), kPAThreads, smem, (cudaStream_t)stream>>>(
       proj, ldp, H, G, M, d, dv, RB, kc, vc, dt_cache, positions, seq_of, pages, max_pages, page_size, scale, chunk, window, out, nsplit,
-      part_acc, part_ml, cu, skip_from, softcap, sinks, pool, pool > 0 ? (page_size + pool - 1) / pool : 0, kp, vp, pool_only);
+      part_acc, part_ml, cu, skip_from, softcap, sinks, pool, pool > 0 ? (page_size + pool - 1) / pool : 0, kp, vp, pool_only, slopes);
   SEQ_LAUNCHED();
   return KB2SEQ_OK;
 }
@@ -870,8 +883,9 @@ KB2SEQ_API int kb2_seq_glu(const void* in, int dt_in, long long ld_in, void* out
 }
 
 KB2SEQ_API int kb2_seq_route(const float* z, long long ldz, int T, int E, const float* correction, int score_kind, int groups, int keep,
-                             int top, int renorm, float out_scale, int* ids, float* weights, int group_kind, void* stream) {
-  if (!z || !ids || !weights || T <= 0 || E <= 0 || top <= 0 || top > E || score_kind < 0 || score_kind > 1 || groups < 1 || group_kind < 0 || group_kind > 1 ||
+                             int top, int renorm, float out_scale, int* ids, float* weights, int group_kind, const float* bias,
+                             void* stream) {
+  if (!z || !ids || !weights || T <= 0 || E <= 0 || top <= 0 || top > E || score_kind < 0 || score_kind > 2 || groups < 1 || group_kind < 0 || group_kind > 1 ||
       E % groups || keep < 1 || keep > groups)
     return failf(KB2SEQ_ERR_VALUE, "route: bad argument (E=%d top=%d groups=%d keep=%d)", E, top, groups, keep);
   if ((long long)keep * (E / groups) < top) return failf(KB2SEQ_ERR_VALUE, "route: the kept groups hold fewer than top experts");
@@ -879,7 +893,7 @@ KB2SEQ_API int kb2_seq_route(const float* z, long long ldz, int T, int E, const 
   if (smem > 200 * 1024) return failf(KB2SEQ_ERR_VALUE, "route: %d router outputs too many", E);
   if (smem > 48 * 1024) SEQ_CUDA(cudaFuncSetAttribute(route_topk_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
   route_topk_kernel<<<(T + 3) / 4, 128, smem, (cudaStream_t)stream>>>(z, ldz, T, E, correction, score_kind, groups, keep, top, renorm,
-                                                                      out_scale, ids, weights, group_kind);
+                                                                      out_scale, ids, weights, group_kind, bias);
   SEQ_LAUNCHED();
   return KB2SEQ_OK;
 }

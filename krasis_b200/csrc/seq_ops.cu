@@ -10,7 +10,8 @@
 //   side_gate              gelu_tanh(g) * per-layer slice of a token table            (per-layer token input)
 //   latent_prep            RMS-normed latent + rotated shared key -> paged cache, rotary on the query's rotated part (any frequency
 //                          table); the latent columns follow the queries or come from a buffer of their own
-//   latent_window_attn     absorbed-form latent attention over the page list: sliding window, softmax with an optional per-head sink
+//   latent_window_attn     absorbed-form latent attention over the page list: sliding window, softmax with an optional per-head sink,
+//                          optional sigmoid gate per head on the result
 //   conv_silu (+ state)    short causal convolution per channel over time with a carried tail, optional bias ahead of the taps or on
 //                          their result, then SiLU or nothing; conv_run reads every input once on long steps
 //   delta_rule             gated delta rule S <- g S; u = beta (v - S^T k); S += k u^T; o = S^T q, state in fp32 slots,
@@ -424,13 +425,17 @@ __global__ void __launch_bounds__(128) latent_prep_kernel(float* __restrict__ pr
 // 0 <= pos - j < window; the softmax denominator also holds exp(sink_h) (a key with no value: running max starts at the sink,
 // running sum at 1).  Output: sum_j p_j c_j (the value up-projection follows as a per-head GEMM).
 // One block per (token, group of HG heads); keys in tiles of KT, shared by the heads of the group.
+// gate [T, ldg] (may be null): head h's output is multiplied by sigmoid(gate[t, h]); it commutes with the value up-projection.
 constexpr int kAttnThreads = 256, kAttnAcc = 16;
+__device__ __forceinline__ float head_gate(const float* __restrict__ gate, long long ldg, long long t, int h) {
+  return gate != nullptr ? 1.f / (1.f + expf(-gate[t * ldg + h])) : 1.f;
+}
 __global__ void __launch_bounds__(kAttnThreads) latent_window_attn_kernel(
     const float* __restrict__ q_abs, const float* __restrict__ proj, long long ldp, int H, int HG, int dn, int dr, int r,
     const void* __restrict__ ckv, const void* __restrict__ kr, int dt_cache, const int* __restrict__ positions,
     const int* __restrict__ seq_of, const int* __restrict__ pages, int max_pages, int page_size, const float* __restrict__ sinks,
     float scale, int window, int KT, float* __restrict__ out, const int* __restrict__ cu, int skip_from, int nsplit,
-    float* __restrict__ part_acc, float* __restrict__ part_ml) {
+    float* __restrict__ part_acc, float* __restrict__ part_ml, const float* __restrict__ gate, long long ldg) {
   extern __shared__ __align__(16) float sm[];
   if (cu != nullptr) {                    // sequences whose portion has skip_from tokens or more are served by another kernel
     const int sq = seq_of[blockIdx.x];
@@ -562,7 +567,7 @@ __global__ void __launch_bounds__(kAttnThreads) latent_window_attn_kernel(
     if (i < nh * r) {
       const int hh = i / r, d = i - hh * r;
       if (nsplit > 1) part_acc[((t * nsplit + z) * H + h0 + hh) * r + d] = acc[a];
-      else out[(t * H + h0 + hh) * r + d] = acc[a] / l_run[hh];
+      else out[(t * H + h0 + hh) * r + d] = acc[a] / l_run[hh] * head_gate(gate, ldg, t, h0 + hh);
     }
   }
   if (nsplit > 1 && tid < nh) {
@@ -574,7 +579,8 @@ __global__ void __launch_bounds__(kAttnThreads) latent_window_attn_kernel(
 // out[t, h, :] = sum_z w_z acc_z / sum_z w_z l_z with w_z = exp(m_z - max_z m_z); pieces without keys have l_z = 0
 __global__ void __launch_bounds__(128) latent_attn_combine_kernel(const float* __restrict__ part_acc, const float* __restrict__ part_ml,
                                                                   int H, int r, int nsplit, float* __restrict__ out,
-                                                                  const int* __restrict__ seq_of, const int* __restrict__ cu, int skip_from) {
+                                                                  const int* __restrict__ seq_of, const int* __restrict__ cu, int skip_from,
+                                                                  const float* __restrict__ gate, long long ldg) {
   const long long t = blockIdx.x;
   const int h = blockIdx.y;
   if (cu != nullptr) {
@@ -597,7 +603,7 @@ __global__ void __launch_bounds__(128) latent_attn_combine_kernel(const float* _
       const float* ml = part_ml + ((t * nsplit + zz) * H + h) * 2;
       if (ml[1] > 0.f) v = fmaf(part_acc[((t * nsplit + zz) * H + h) * r + d], expf(ml[0] - M), v);
     }
-    out[(t * H + h) * r + d] = v / L;
+    out[(t * H + h) * r + d] = v / L * head_gate(gate, ldg, t, h);
   }
 }
 
@@ -1080,7 +1086,7 @@ KB2SEQ_API int kb2_seq_latent_window_attn(const float* q_abs, const float* proj,
                                           const void* ckv, const void* kr, int dt_cache, const int* positions, const int* seq_of,
                                           const int* pages, int max_pages, int page_size, const float* sinks, float scale, int window,
                                           float* out, const int* cu, int skip_from, int nsplit, float* part_acc, float* part_ml,
-                                          void* stream) {
+                                          const float* gate, long long ldg, void* stream) {
   if (!q_abs || !proj || !ckv || !kr || !positions || !seq_of || !pages || !out || T <= 0 || H <= 0 || r <= 0 || dr < 0 ||
       window <= 0 || bad_dt(dt_cache))
     return failf(KB2SEQ_ERR_VALUE, "latent_window_attn: bad argument");
@@ -1098,10 +1104,10 @@ KB2SEQ_API int kb2_seq_latent_window_attn(const float* q_abs, const float* proj,
   dim3 grid(T, (H + HG - 1) / HG, nsplit);
   latent_window_attn_kernel<<<grid, kAttnThreads, smem, (cudaStream_t)stream>>>(q_abs, proj, ldp, H, HG, dn, dr, r, ckv, kr, dt_cache, positions,
                                                                                  seq_of, pages, max_pages, page_size, sinks, scale, window, KT,
-                                                                                 out, cu, skip_from, nsplit, part_acc, part_ml);
+                                                                                 out, cu, skip_from, nsplit, part_acc, part_ml, gate, ldg);
   SEQ_LAUNCHED();
   if (nsplit > 1) {
-    latent_attn_combine_kernel<<<dim3(T, H), 128, 0, (cudaStream_t)stream>>>(part_acc, part_ml, H, r, nsplit, out, seq_of, cu, skip_from);
+    latent_attn_combine_kernel<<<dim3(T, H), 128, 0, (cudaStream_t)stream>>>(part_acc, part_ml, H, r, nsplit, out, seq_of, cu, skip_from, gate, ldg);
     SEQ_LAUNCHED();
   }
   return KB2SEQ_OK;

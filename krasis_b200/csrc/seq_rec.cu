@@ -1,5 +1,5 @@
 // Ragged-batch sequence operators, third part: linear recurrences with per-sequence state slots and the small row kernels of
-// designs that run several mixers side by side or average their residual stream over depth.
+// designs that run several mixers side by side, average their residual stream over depth or keep several copies of it.
 //
 //   gla_scan / gla_reg     gated linear attention, S <- diag(alpha_t) S + k_t v_t^T, o_t = S^T q_t per head, with one decay per key
 //                          channel alpha = sigmoid(z)^(1 / tau); the state of a (sequence, head, slice of value columns) lives in
@@ -12,6 +12,8 @@
 //   branch_merge           c (a / rms(a) * wa + b / rms(b) * wb): two mixers that read the same input, each normed, averaged
 //   depth_mix              the residual stream as a learned weighted sum of the embedding output and every layer's result, fused with
 //                          the residual add that completes the newest result and with the next norm
+//   stream_mix             several copies of the residual stream: every copy becomes a weighted sum of all copies plus a share of the
+//                          sublayer's output, fused with the weighted sum the next sublayer reads and with its norm
 //
 // Precision: decays, step sizes, softplus / exponentials, states, norms and every accumulation are fp32; `dt` selects storage only.
 #include "seq_common.cuh"
@@ -395,6 +397,115 @@ __global__ void __launch_bounds__(256) depth_mix_kernel(float* __restrict__ stac
   for (int i = threadIdx.x; i < W; i += blockDim.x) st_dt(h, dt_h, t * W + i, xr[i] * rstd * w[i]);
 }
 
+// xs [T][n][W]: n copies of the residual stream per token, one block per token.  A thread keeps its columns of all copies in registers, so
+// the copies are read and written once; the row of u waits in shared memory for the norm.  NS: the number of copies (0: n, up to 32);
+// V: columns per access (4 needs W % 4 == 0 and 16-byte rows).
+constexpr int kMaxStreams = 32;
+template <int V> struct Cols { float v[V]; };
+template <int V> __device__ __forceinline__ Cols<V> ld_cols(const float* p) {
+  Cols<V> c;
+  if constexpr (V == 4) {
+    const float4 f = *reinterpret_cast<const float4*>(p);
+    c.v[0] = f.x; c.v[1] = f.y; c.v[2] = f.z; c.v[3] = f.w;
+  } else {
+    c.v[0] = p[0];
+  }
+  return c;
+}
+template <int V> __device__ __forceinline__ void st_cols(float* p, const Cols<V>& c) {
+  if constexpr (V == 4) *reinterpret_cast<float4*>(p) = make_float4(c.v[0], c.v[1], c.v[2], c.v[3]);
+  else p[0] = c.v[0];
+}
+template <int NS, int V>
+__global__ void __launch_bounds__(256) stream_mix_kernel(float* __restrict__ xs, int n_rt, const float* __restrict__ x0,
+                                                         const float* __restrict__ y, const float* __restrict__ mix,
+                                                         const float* __restrict__ out, const float* __restrict__ read,
+                                                         const float* __restrict__ w, float w_shift, void* __restrict__ h, int dt_h, int W,
+                                                         float eps) {
+  constexpr int N = NS > 0 ? NS : kMaxStreams, U = NS > 0 ? NS : 1;      // the generic form keeps its loops over the copies rolled
+  extern __shared__ __align__(16) float u_row[];           // [W]
+  __shared__ float cm[N * N], co[N], cr[N], red[32];
+  const int n = NS > 0 ? NS : n_rt;
+  const long long t = blockIdx.x;
+  for (int i = threadIdx.x; i < n * n; i += blockDim.x) cm[i] = y != nullptr ? mix[i] : 0.f;
+  for (int i = threadIdx.x; i < n; i += blockDim.x) {
+    co[i] = y != nullptr ? out[i] : 0.f;
+    cr[i] = read != nullptr ? read[i] : 1.f;
+  }
+  __syncthreads();
+  float* xt = xs + t * n * W;
+  float ss = 0.f;
+  for (int d = threadIdx.x * V; d < W; d += blockDim.x * V) {
+    Cols<V> x[N], u;
+    if (x0 != nullptr) {
+      const Cols<V> e = ld_cols<V>(x0 + t * W + d);
+#pragma unroll U
+      for (int s = 0; s < N; ++s) if (s < n) x[s] = e;
+    } else {
+#pragma unroll U
+      for (int s = 0; s < N; ++s) if (s < n) x[s] = ld_cols<V>(xt + (long long)s * W + d);
+    }
+#pragma unroll
+    for (int c = 0; c < V; ++c) u.v[c] = 0.f;
+    if (y != nullptr) {
+      const Cols<V> yv = ld_cols<V>(y + t * W + d);
+#pragma unroll U
+      for (int q = 0; q < N; ++q) {
+        if (q < n) {
+          Cols<V> r;
+#pragma unroll
+          for (int c = 0; c < V; ++c) r.v[c] = 0.f;
+#pragma unroll U
+          for (int s = 0; s < N; ++s)
+            if (s < n) {
+#pragma unroll
+              for (int c = 0; c < V; ++c) r.v[c] = fmaf(cm[s * n + q], x[s].v[c], r.v[c]);
+            }
+#pragma unroll
+          for (int c = 0; c < V; ++c) {
+            r.v[c] = fmaf(co[q], yv.v[c], r.v[c]);
+            u.v[c] = fmaf(cr[q], r.v[c], u.v[c]);
+          }
+          st_cols<V>(xt + (long long)q * W + d, r);
+        }
+      }
+    } else {
+#pragma unroll U
+      for (int s = 0; s < N; ++s)
+        if (s < n) {
+#pragma unroll
+          for (int c = 0; c < V; ++c) u.v[c] = fmaf(cr[s], x[s].v[c], u.v[c]);
+          if (x0 != nullptr) st_cols<V>(xt + (long long)s * W + d, x[s]);
+        }
+    }
+    st_cols<V>(u_row + d, u);
+#pragma unroll
+    for (int c = 0; c < V; ++c) ss = fmaf(u.v[c], u.v[c], ss);
+  }
+  if (h == nullptr) return;
+  float rstd = 1.f;
+  if (w != nullptr) rstd = 1.f / sqrtf(block_sum(ss, red) / (float)W + eps);
+  for (int d = threadIdx.x * V; d < W; d += blockDim.x * V) {       // a thread reads back the columns it wrote
+    Cols<V> u = ld_cols<V>(u_row + d);
+    if (w != nullptr) {
+      const Cols<V> wv = ld_cols<V>(w + d);
+#pragma unroll
+      for (int c = 0; c < V; ++c) u.v[c] = u.v[c] * rstd * (w_shift + wv.v[c]);
+    }
+    if (dt_h == 0) {
+      st_cols<V>((float*)h + t * W + d, u);
+    } else if constexpr (V == 4) {
+      const __nv_bfloat162 lo = __floats2bfloat162_rn(u.v[0], u.v[1]), hi = __floats2bfloat162_rn(u.v[2], u.v[3]);
+      uint2 o;
+      o.x = *reinterpret_cast<const uint32_t*>(&lo);
+      o.y = *reinterpret_cast<const uint32_t*>(&hi);
+      *reinterpret_cast<uint2*>((bf16*)h + t * W + d) = o;
+    } else {
+      ((bf16*)h)[t * W + d] = __float2bfloat16_rn(u.v[0]);
+    }
+  }
+}
+
 static int pow2_at_least(int v) {
   int p = 1;
   while (p < v) p <<= 1;
@@ -512,6 +623,34 @@ KB2SEQ_API int kb2_seq_depth_mix(float* stack, long long stride, int n, const fl
                                  int dt_h, int T, int W, float eps, void* stream) {
   if (!stack || !coef || !x || n <= 0 || T <= 0 || W <= 0 || (w && (!h || bad_dt(dt_h)))) return failf(KB2SEQ_ERR_VALUE, "depth_mix: bad argument");
   depth_mix_kernel<<<T, 256, 0, (cudaStream_t)stream>>>(stack, stride, n, coef, x, y, w, h, dt_h, W, eps);
+  SEQ_LAUNCHED();
+  return KB2SEQ_OK;
+}
+
+KB2SEQ_API int kb2_seq_stream_mix(float* xs, int n, const float* x0, const float* y, const float* mix, const float* out, const float* read,
+                                  const float* w, float w_shift, void* h, int dt_h, int T, int W, float eps, void* stream) {
+  if (!xs || n < 1 || n > kMaxStreams || T <= 0 || W <= 0 || (y && (!mix || !out)) || (w && !h) || (h && bad_dt(dt_h)))
+    return failf(KB2SEQ_ERR_VALUE, "stream_mix: bad argument (n=%d T=%d W=%d)", n, T, W);
+  const size_t smem = (size_t)W * 4;
+  if (smem > 200 * 1024) return failf(KB2SEQ_ERR_VALUE, "stream_mix: width %d too large", W);
+  const uintptr_t all = (uintptr_t)xs | (uintptr_t)x0 | (uintptr_t)y | (uintptr_t)w | (uintptr_t)h;
+  const bool vec = W % 4 == 0 && !(all & 15);
+  cudaStream_t s = (cudaStream_t)stream;
+#define KB2_SM(NSV, VV)                                                                                                              \
+  do {                                                                                                                               \
+    if (smem > 40 * 1024) SEQ_CUDA(cudaFuncSetAttribute(stream_mix_kernel<NSV, VV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); \
+    stream_mix_kernel<NSV, VV><<<T, 256, smem, s>>>(xs, n, x0, y, mix, out, read, w, w_shift, h, dt_h, W, eps);                      \
+  } while (0)
+  if (!vec) KB2_SM(0, 1);
+  else switch (n) {
+    case 1: KB2_SM(1, 4); break;
+    case 2: KB2_SM(2, 4); break;
+    case 3: KB2_SM(3, 4); break;
+    case 4: KB2_SM(4, 4); break;
+    case 8: KB2_SM(8, 4); break;
+    default: KB2_SM(0, 1); break;
+  }
+#undef KB2_SM
   SEQ_LAUNCHED();
   return KB2SEQ_OK;
 }

@@ -34,7 +34,7 @@ import torch
 
 from . import seqops as ops
 from .attention import HeadKVCache, RecurrentStatePool
-from .mixers import ChannelDeltaMixer, GatedMLP, MultiMapAttention, RoutedExperts, lin, llama3_table
+from .mixers import ChannelDeltaMixer, GatedMLP, MultiMapAttention, RoutedExperts, layer_runs, lin, llama3_table
 
 NORM_SHIFT = 1.0          # a norm's weight tensor holds the offset from one
 GROUP_MEMBERS = "top2"    # an expert group competes with its best two members added up
@@ -79,13 +79,7 @@ class GurozenConfig:
 
     def runs(self):
         """[(layer index, True if a pass of the looped span starts with this run)] in execution order."""
-        n = len(self.layers)
-        if not self.has_loop:
-            return [(i, False) for i in range(n)]
-        out = [(i, False) for i in range(self.loop_start)]
-        for _ in range(self.loop_times):
-            out += [(i, i == self.loop_start) for i in range(self.loop_start, self.loop_stop)]
-        return out + [(i, False) for i in range(self.loop_stop, n)]
+        return layer_runs(len(self.layers), self.loop_start, self.loop_stop, self.loop_times)
 
 
 def _sub(weights: dict, prefix: str) -> dict:

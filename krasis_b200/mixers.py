@@ -5,7 +5,7 @@ libkrasis_b200_seq (`krasis_b200.seqops`): a model composes them (krasis_b200/vo
 
   WindowLatentAttention   attention over a cached low-rank latent with one shared rotated key part, interleaved rotary positions
                           with YaRN frequency blending, a sliding window and a per-head softmax sink (optional: queries through a
-                          normed latent of their own, no sink, a sigmoid output gate per element)
+                          normed latent of their own, no sink, a sigmoid output gate per element or per head)
   GatedDeltaMixer         short causal convolutions on q / k / v, unit-norm q and k, gated delta-rule state per head in fp32
                           slots, per-head RMS norm of the read-out with a SiLU gate
   MultiMapAttention       grouped-query attention over a per-head paged cache whose heads carry several attention maps (keys per
@@ -16,7 +16,8 @@ libkrasis_b200_seq (`krasis_b200.seqops`): a model composes them (krasis_b200/vo
                           (further options: a short causal convolution on q / k / v after the projection, one RMS norm over the whole
                           of q and of k, rotation of dimension i with i + dims / 2, a frequency table of the caller, tanh soft-capped
                           scores, a softmax sink per head, mean-pooled blocks of keys and values before the window, values cached
-                          rotated by their positions with the output turned back, an output gate per element)
+                          rotated by their positions with the output turned back, an output gate per element, query and key norms
+                          without weights, a penalty per head that grows with the distance to the key)
   GatedLinearAttention    S <- diag(alpha) S + k v^T with one decay per key channel, alpha = sigmoid(.)^(1 / tau) from a low-rank
                           projection; per-head RMS norm of the read-out with a SiLU gate
   SelectiveScan           Mamba: input / gate projection, short causal convolution, input-dependent step sizes and B / C, diagonal
@@ -27,8 +28,9 @@ libkrasis_b200_seq (`krasis_b200.seqops`): a model composes them (krasis_b200/vo
   GatedMLP                down(act(gate h) * (up h)): tanh-GELU, SiLU, or the clamped swish form g' sigmoid(a g') (u' + 1); without a
                           gate: down(relu(up h)^2)
   RoutedExperts           softmax / sigmoid router with a choice correction, expert groups (scored by their best or their two best
-                          outputs) and identity experts, top-k experts of either form (binned tile GEMMs; a GEMV form for steps of few
-                          tokens) plus an optional shared expert with an optional per-token sigmoid gate
+                          outputs) and identity experts, or a choice by the biased logits with a softmax over the chosen ones; top-k
+                          experts of any of those forms (binned tile GEMMs; a GEMV form for steps of few tokens) plus an optional shared
+                          expert with an optional per-token sigmoid gate
   TokenSideInput          per-layer token table slice, gated by a projection of the residual stream, RMS-normed
 `lin(a, w, out_dtype)` picks the GEMM: the tcgen05 kernel of the core library for large aligned bf16 products, the generic
 kernel of the sequence library otherwise (any shape, fp32 or bf16).
@@ -76,6 +78,15 @@ def lin(a: torch.Tensor, w: torch.Tensor, out_dtype=torch.float32, min_n: int = 
     return ops.gemm(a, w, out_dtype)
 
 
+def layer_runs(n: int, start: int = 0, stop: int = 0, times: int = 1):
+    """[(layer index, True if a pass of the looped span starts with this run)] in execution order: layers start .. stop - 1 run `times`
+    times in a row, the others once.  No span (stop <= start, or times < 1): every layer once."""
+    if times < 1 or stop <= start:
+        return [(i, False) for i in range(n)]
+    return ([(i, False) for i in range(start)] + [(i, i == start) for _ in range(times) for i in range(start, stop)]
+            + [(i, False) for i in range(stop, n)])
+
+
 def yarn_table(dims: int, base: float, scaling):
     """Angular frequency of each rotated pair (fp64) and the amplitude both sin and cos carry.
     scaling = {factor, original, fast, slow} or None: pairs that turn more than `fast` times over `original` positions keep their
@@ -98,7 +109,8 @@ def yarn_table(dims: int, base: float, scaling):
 class WindowLatentAttention:
     """weights: q [H (dn + dr), W], dkv [r + dr, W], dkv_norm [r], uk [H dn, r], uv [H dv, r], sink [H] (optional), o [W, H dv].
     Instead of q: dq [rq, W], dq_norm [rq], uq [H (dn + dr), rq] — queries from an RMS-normed latent of their own.
-    g [H dv, W] (optional): the concatenated heads are multiplied by sigmoid(g h) ahead of the output projection.
+    g (optional): the concatenated heads are multiplied by sigmoid(g h) ahead of the output projection, one gate per element
+    (g [H dv, W]) or one per head (g [H, W]).
     rot_freq: the frequency table (fp64, one per rotated pair), if not the YaRN table of rot_base / rot_scaling."""
 
     def __init__(self, weights: dict, heads: int, dim: int, rot_dim: int, vdim: int, kv_rank: int, scale: float, window,
@@ -119,10 +131,16 @@ class WindowLatentAttention:
         first = weights["dq"] if self.q_latent else weights["q"]
         self.q_cols = first.shape[0]                                               # q itself, or the query latent
         rows = [first, weights["dkv"]]
-        self.gate_off = -1
+        self.gate_off, self.gate_wide = -1, False
         if "g" in weights:
             self.gate_off = self.q_cols + kv_rank + rot_dim
             rows.append(weights["g"])
+            self.gate_wide = weights["g"].shape[0] == heads * vdim
+            if weights["g"].shape[0] not in (heads, heads * vdim):
+                raise ValueError("output gate: one row per head or per element")
+            pad = 0 if self.gate_wide else -sum(r.shape[0] for r in rows) % 16      # a width the tensor-core product takes
+            if pad:
+                rows.append(torch.zeros(pad, first.shape[1], dtype=first.dtype))
         self.w_in = d(torch.cat(rows, 0))                                          # one projection: [q | latent | rotated key | gate]
         if self.q_latent:
             self.dq_norm, self.w_uq = f(weights["dq_norm"]), d(weights["uq"])
@@ -156,7 +174,9 @@ class WindowLatentAttention:
                                           tb.pages.data_ptr(), tb.max_pages, page_size, ckv.data_ptr(), kr.data_ptr(), dtc, ops._ptr(lat),
                                           proj_in.stride(0), s))
         q = proj[:, :H * (self.dn + self.dr)].view(T, H, self.dn + self.dr)
-        gated = self.gate_off >= 0
+        gated = self.gate_off >= 0 and self.gate_wide                          # per element: a pass over the heads' outputs
+        hg = proj_in[:, self.gate_off:] if self.gate_off >= 0 and not self.gate_wide else None    # per head: inside the attention kernels
+        ldg = proj_in.stride(0)
         o = torch.empty((T, H, self.dv), dtype=torch.float32 if gated else self.dtype, device=h.device)
         core = _core_lib() if self.tc_shape else False
         fast = [i for i, (_, n, _, _) in enumerate(tb.layout) if n >= self.tc_min_portion] if core else []
@@ -175,7 +195,7 @@ class WindowLatentAttention:
                                                      tb.max_pages, page_size, ops._ptr(self.sink), self.scale, self.window,
                                                      o_lat.data_ptr(), tb.cu.data_ptr() if fast else None, self.tc_min_portion, nsplit,
                                                      part_acc.data_ptr() if nsplit > 1 else None,
-                                                     part_ml.data_ptr() if nsplit > 1 else None, s))
+                                                     part_ml.data_ptr() if nsplit > 1 else None, ops._ptr(hg), ldg, s))
             ops.gemm_heads(o_lat, self.uv, o)
         for i in fast:
             from . import capi
@@ -185,9 +205,9 @@ class WindowLatentAttention:
             kpe = kr.view(-1, self.dr).index_select(0, rows)
             q_bf = proj[row0:row0 + n, :H * (self.dn + self.dr)].to(torch.bfloat16).contiguous()
             o_rows = torch.empty((n, H, self.dv), dtype=torch.bfloat16, device=h.device) if gated else o[row0:row0 + n]
-            capi.check(core.kb2_fmha_latent(q_bf.data_ptr(), kv_up.data_ptr(), kpe.data_ptr(), o_rows.data_ptr(), n, start - lo,
-                                            start - lo + n, H, self.scale, min(self.window, 1 << 30), ops._ptr(self.sink),
-                                            h.device.index or 0, s))
+            capi.check(core.kb2_fmha_latent_gated(q_bf.data_ptr(), kv_up.data_ptr(), kpe.data_ptr(), o_rows.data_ptr(), n, start - lo,
+                                                  start - lo + n, H, self.scale, min(self.window, 1 << 30), ops._ptr(self.sink),
+                                                  hg[row0:].data_ptr() if hg is not None else None, ldg, h.device.index or 0, s))
             if gated:
                 o[row0:row0 + n].copy_(o_rows)
         if gated:
@@ -451,6 +471,12 @@ def llama3_table(dims: int, base: float, scaling=None) -> torch.Tensor:
     return torch.where(wave < orig / high, f, torch.where(wave > orig / low, f / factor, mid))
 
 
+def distance_slopes(heads: int) -> torch.Tensor:
+    """Slope of head h's distance penalty (fp64): 2^(-8 (h + 1) / heads), a geometric series that ends at 2^-8 (the slopes of
+    Press, Smith and Lewis, "Train Short, Test Long: Attention with Linear Biases Enables Input Length Extrapolation")."""
+    return torch.pow(torch.tensor(2.0, dtype=torch.float64), -8.0 * torch.arange(1, heads + 1, dtype=torch.float64) / heads)
+
+
 class MultiMapAttention:
     """weights: q [H M d, W], k [G M d, W], v [G dv, W] (each with an optional bias `<name>_b`), q_norm / k_norm [d] (optional RMS norm
     weights, shared by heads and maps), g [H, W] (optional output gate), o [W, H dv].  Rows of q and k are laid out head by head as
@@ -471,13 +497,15 @@ class MultiMapAttention:
     before its window — the means of the block's cached keys and values, kept in pooled pools (`forward(..., pooled=(kp, vp))`).
     rot_values: values are cached rotated by their positions over all of vdim (pair m by position * rot_base^(-2m / vdim), no factor,
     the pair layout of the keys) and each head's output is turned back by the query's position, ahead of the gate.
-    gate_per_element: g is [H dv, W], one sigmoid gate per output element (default [H, W]: one per head)."""
+    gate_per_element: g is [H dv, W], one sigmoid gate per output element (default [H, W]: one per head).
+    qk_unit: every query and key vector is divided by its root mean square, without a weight.
+    slopes [H]: slopes[h] times the distance (query position - key position) is taken off head h's scores, after scale and cap."""
 
     def __init__(self, weights: dict, heads: int, kv_heads: int, maps: int, dim: int, vdim: int, scale: float, eps: float, dtype, device,
                  chunk=None, window=None, rot_dims: int = 0, rot_base: float = 10000.0, rot_factor: float = 1.0, map_coef=None,
                  unit_norm: bool = False, post_scale: float = 1.0, own_kv: bool = True, conv_taps: int = 0, norm_whole: bool = False,
                  rot_half: bool = False, rot_freq=None, softcap: float = 0.0, pool: int = 0, rot_values: bool = False,
-                 gate_per_element: bool = False):
+                 gate_per_element: bool = False, qk_unit: bool = False, slopes=None):
         if heads % kv_heads:
             raise ValueError("heads must be a multiple of kv_heads")
         if rot_dims > dim or rot_dims % 2:
@@ -522,6 +550,15 @@ class MultiMapAttention:
             self.bias = None
         self.q_norm = f(weights["q_norm"]) if "q_norm" in weights else None
         self.k_norm = f(weights["k_norm"]) if (own_kv and "k_norm" in weights) else None
+        if qk_unit:
+            if norm_whole or self.q_norm is not None or self.k_norm is not None:
+                raise ValueError("unit queries and keys have no norm weights")
+            self.q_norm = torch.ones(dim, dtype=torch.float32, device=device)
+            self.k_norm = torch.ones(dim, dtype=torch.float32, device=device) if own_kv else None
+        self.slopes = f(torch.as_tensor(slopes)) if slopes is not None else None
+        if self.slopes is not None and (self.slopes.numel() != heads or self.pool):
+            raise ValueError("one slope per head, and no pooled blocks beside them")
+        self.map_slopes = self.slopes.repeat_interleave(self.M).contiguous() if self.slopes is not None else None    # per query vector
         self.w_o = d(weights["o"])
         self.C = sum(weights[n].shape[0] for n in names)                    # q | k | v columns of the projection
         self.taps = f(torch.cat([weights[n + "_conv"] for n in names], 0)) if self.K else None
@@ -565,7 +602,12 @@ class MultiMapAttention:
             end = min(start + n, cstart + chunk) if chunk else start + n
             lo = max(cstart, first)
             m = end - pos
-            if self.sink is not None or lse is not None:
+            if self.slopes is not None:
+                capi.check(core.kb2_fmha_maps_slopes(q[pos - start:].data_ptr(), k_rows[lo - first:].data_ptr(), v_rows[lo - first:].data_ptr(),
+                                                     a[row0 + pos - start:].data_ptr(), m, pos - lo, end - lo, H * M, G, M, dv, self.scale,
+                                                     self.softcap, min(self.window, 1 << 30), ops._ptr(self.sink), None,
+                                                     self.map_slopes.data_ptr(), proj.device.index or 0, stream))
+            elif self.sink is not None or lse is not None:
                 capi.check(core.kb2_fmha_maps_sink(q[pos - start:].data_ptr(), k_rows[lo - first:].data_ptr(), v_rows[lo - first:].data_ptr(),
                                                    a[row0 + pos - start:].data_ptr(), m, pos - lo, end - lo, H * M, G, M, dv, self.scale,
                                                    self.softcap, min(self.window, 1 << 30), ops._ptr(self.sink),
@@ -616,7 +658,7 @@ class MultiMapAttention:
                                              tb.positions.data_ptr(), tb.seq_of.data_ptr(), tb.pages.data_ptr(), tb.max_pages, page_size,
                                              self.scale, self.chunk, min(self.window, 1 << 30), a.data_ptr(), nsplit, ops._ptr(part_acc),
                                              ops._ptr(part_ml), tb.cu.data_ptr() if fast else None, self.tc_min_portion, self.softcap,
-                                             ops._ptr(self.sink), self.pool, ops._ptr(kp), ops._ptr(vp), 0, s))
+                                             ops._ptr(self.sink), self.pool, ops._ptr(kp), ops._ptr(vp), 0, ops._ptr(self.slopes), s))
         lse = torch.empty((T, H), dtype=torch.float32, device=h.device) if (fast and self.pool) else None
         for i in fast:
             self._tensor_core_portion(core, proj, a, tb, i, kc, vc, page_size, s, lse=lse)
@@ -627,7 +669,7 @@ class MultiMapAttention:
                                              tb.positions.data_ptr(), tb.seq_of.data_ptr(), tb.pages.data_ptr(), tb.max_pages, page_size,
                                              self.scale, 0, min(self.window, 1 << 30), a.data_ptr(), 1, p_acc.data_ptr(), p_ml.data_ptr(),
                                              tb.cu.data_ptr(), self.tc_min_portion, self.softcap, None, self.pool, kp.data_ptr(),
-                                             vp.data_ptr(), 1, s))
+                                             vp.data_ptr(), 1, None, s))
             ops.check(lib.kb2_seq_pool_merge(a.data_ptr(), lse.data_ptr(), p_acc.data_ptr(), p_ml.data_ptr(), T, H, self.dv,
                                              tb.seq_of.data_ptr(), tb.cu.data_ptr(), self.tc_min_portion, s))
         o = torch.empty((T, H * self.dv), dtype=self.dtype, device=h.device)
@@ -643,7 +685,10 @@ class RoutedExperts:
     """weights: router [E + identity, W], correction [E + identity] (optional), e<i>_gate / e<i>_up [F, W], e<i>_down [W, F] for i < E,
     shared_gate / shared_up / shared_down (optional shared expert of the same form, run for every token and added), shared_sg [1, W]
     (optional: the shared expert's output is multiplied by sigmoid(shared_sg h), one number per token).
-    gated False: the experts (and the shared one) have no gate tensor and compute down(act(up h)); act: "silu" (gated) or "relu2".
+    gated False: the experts (and the shared one) have no gate tensor and compute down(act(up h)); act: "silu" or "clamped_swish" (gated,
+    with limit and alpha as in GatedMLP; shared_limit: the shared expert's own limit) or "relu2" (no gate).
+    router_b [E + identity] (optional) is added to the router logits in fp32.  score "top_softmax": the largest logits are chosen, and
+    the weights are the softmax over the chosen logits alone.
 
     Scores are softmax (or sigmoid) of the fp32 router logits over all E + identity outputs; the choice adds `correction`; the outputs
     form `groups` equal groups of neighbours of which the `keep` with the largest group score stay eligible (group_score "max": the
@@ -652,14 +697,16 @@ class RoutedExperts:
 
     def __init__(self, weights: dict, experts: int, identity: int, top: int, dtype, device, groups: int = 1, keep: int = 1,
                  score: str = "softmax", renorm: bool = False, out_scale: float = 1.0, gated: bool = True, act: str = "silu",
-                 group_score: str = "max"):
+                 group_score: str = "max", limit: float = 0.0, alpha: float = 1.0, shared_limit=None):
         d = lambda t: t.to(device=device, dtype=dtype).contiguous()
         self.E, self.ident, self.top, self.groups, self.keep = int(experts), int(identity), int(top), int(groups), int(keep)
         self.score, self.renorm, self.out_scale, self.dtype, self.device = score, bool(renorm), float(out_scale), dtype, device
         self.gated, self.group_score = bool(gated), group_score
-        if gated == (act == "relu2") or act not in ("silu", "relu2") or group_score not in ("max", "top2"):
-            raise ValueError("experts: silu with a gate or relu2 without; group_score max or top2")
-        self.act_kind = ops.GLU_SILU if gated else ops.ACT_RELU2
+        if gated == (act == "relu2") or act not in ("silu", "clamped_swish", "relu2") or group_score not in ("max", "top2"):
+            raise ValueError("experts: silu or clamped_swish with a gate or relu2 without; group_score max or top2")
+        if score not in ops.ROUTE_SCORES:
+            raise ValueError(f"router score {score!r}")
+        self.act_kind, self.limit, self.alpha = GatedMLP.KINDS[act], float(limit), float(alpha)
         if weights["router"].shape[0] != self.E + self.ident:
             raise ValueError("router rows must equal experts + identity experts")
         if (self.E + self.ident) % self.groups or not 1 <= self.keep <= self.groups:
@@ -674,13 +721,17 @@ class RoutedExperts:
                 rows.append(torch.zeros(pad, weights["router"].shape[1], dtype=weights["router"].dtype))
         self.w_router = d(torch.cat(rows, 0))
         self.correction = weights["correction"].to(device=device, dtype=torch.float32).contiguous() if "correction" in weights else None
+        self.router_bias = weights["router_b"].to(device=device, dtype=torch.float32).contiguous() if "router_b" in weights else None
+        if self.router_bias is not None and self.router_bias.numel() != self.E + self.ident:
+            raise ValueError("one router bias per router row")
         if self.E:
             first = (lambda i: torch.cat([weights[f"e{i}_gate"], weights[f"e{i}_up"]], 0)) if gated else (lambda i: weights[f"e{i}_up"])
             self.w_gu = d(torch.stack([first(i) for i in range(self.E)], 0))                         # [E, 2F | F, W]
             self.w_down = d(torch.stack([weights[f"e{i}_down"] for i in range(self.E)], 0))          # [E, W, F]
             self.F = self.w_down.shape[2]
         self.shared = GatedMLP({k[len("shared_"):]: v for k, v in weights.items() if k.startswith("shared_") and k != "shared_sg"}, dtype,
-                               device, act=act, gated=gated) if "shared_up" in weights else None
+                               device, act=act, gated=gated, limit=limit if shared_limit is None else shared_limit,
+                               alpha=alpha) if "shared_up" in weights else None
         self.tile = ops.load().kb2_seq_moe_tile_rows()
         self.gemv_max_tokens = 8
         # bfloat16 steps that bring at least this many rows per expert on average run on the grouped tcgen05 GEMM (128-row tiles)
@@ -720,7 +771,7 @@ class RoutedExperts:
         gu = torch.empty((rows, F1), dtype=torch.bfloat16, device=dev)
         capi.check(core.kb2_linear_bf16_grouped(xs.data_ptr(), self.w_gu.data_ptr(), gu.data_ptr(), rows, F1, W, 0, t["tile_expert"].data_ptr(),
                                                 t["n_tiles"].data_ptr(), E, di, s))
-        act = ops.glu(gu, torch.bfloat16, self.act_kind, n_tiles=t["n_tiles"], tile_rows=128)
+        act = ops.glu(gu, torch.bfloat16, self.act_kind, self.limit, self.alpha, n_tiles=t["n_tiles"], tile_rows=128)
         y = torch.empty((rows, W), dtype=torch.float32, device=dev)
         capi.check(core.kb2_linear_bf16_grouped(act.data_ptr(), self.w_down.data_ptr(), y.data_ptr(), rows, W, F, 1, t["tile_expert"].data_ptr(),
                                                 t["n_tiles"].data_ptr(), E, di, s))
@@ -730,7 +781,7 @@ class RoutedExperts:
         """(ids, weights, router product [T, >= E + identity] whose column sg_col is the shared expert's gate input)."""
         z = lin(h, self.w_router, torch.float32, min_n=16)
         return ops.route(z, self.correction, self.top, self.groups, self.keep, self.score, self.renorm, self.out_scale, self.group_score,
-                         experts=self.E + self.ident) + (z,)
+                         experts=self.E + self.ident, bias=self.router_bias) + (z,)
 
     def forward(self, h: torch.Tensor) -> torch.Tensor:
         lib, T, W, E, top = ops.load(), h.shape[0], h.shape[1], self.E, self.top
@@ -744,7 +795,7 @@ class RoutedExperts:
             gu = torch.empty((slots, F2), dtype=dt, device=dev)
             ops.check(lib.kb2_seq_moe_gemv(h.data_ptr(), ops.dt_code(h.dtype), h.stride(0), top, ids.data_ptr(), E, self.w_gu.data_ptr(), dtc, W,
                                            F2 * W, gu.data_ptr(), dtc, F2, slots, F2, W, s))
-            act = ops.glu(gu, dt, self.act_kind)
+            act = ops.glu(gu, dt, self.act_kind, self.limit, self.alpha)
             y = torch.empty((slots, W), dtype=torch.float32, device=dev)
             ops.check(lib.kb2_seq_moe_gemv(act.data_ptr(), dtc, self.F, 1, ids.data_ptr(), E, self.w_down.data_ptr(), dtc, self.F, W * self.F,
                                            y.data_ptr(), 0, W, slots, W, self.F, s))
@@ -757,7 +808,7 @@ class RoutedExperts:
             gu = torch.empty((max_rows, F2), dtype=dt, device=dev)
             ops.check(lib.kb2_seq_moe_gemm(h.data_ptr(), ops.dt_code(h.dtype), h.stride(0), slot_row.data_ptr(), top, self.w_gu.data_ptr(), dtc, W,
                                            F2 * W, gu.data_ptr(), dtc, F2, F2, W, tile_expert.data_ptr(), n_tiles.data_ptr(), max_tiles, tile, s))
-            act = ops.glu(gu, dt, self.act_kind, n_tiles=n_tiles, tile_rows=tile)
+            act = ops.glu(gu, dt, self.act_kind, self.limit, self.alpha, n_tiles=n_tiles, tile_rows=tile)
             y = torch.empty((max_rows, W), dtype=torch.float32, device=dev)
             ops.check(lib.kb2_seq_moe_gemm(act.data_ptr(), dtc, self.F, None, 1, self.w_down.data_ptr(), dtc, self.F, W * self.F, y.data_ptr(), 0,
                                            W, W, self.F, tile_expert.data_ptr(), n_tiles.data_ptr(), max_tiles, tile, s))

@@ -45,6 +45,13 @@ def _zaronex(model_dir, dtype=torch.bfloat16, device=0, **kw):
     return ZaronexModel.from_pretrained(model_dir, dtype=dtype, device=device, **kw)
 
 
+def _kugalorn(model_dir, dtype=torch.bfloat16, device=0, **kw):
+    from .build import build_seq
+    build_seq()
+    from .kugalorn import KugalornModel
+    return KugalornModel.from_pretrained(model_dir, dtype=dtype, device=device, **kw)
+
+
 def _hf_moe(model_dir, dtype=torch.bfloat16, device=0, **kw):
     if dtype != torch.bfloat16:
         raise ValueError("the MoE prefill models run in bfloat16 only")
@@ -58,6 +65,7 @@ register("Vofelix", _vofelix)
 register("Megolorn", _megolorn)
 register("Gurozen", _gurozen)
 register("Zaronex", _zaronex)
+register("Kugalorn", _kugalorn)
 for _name in _HF_MOE:
     register(_name, _hf_moe)
 

@@ -22,7 +22,7 @@ SIGNATURES = {
     "kb2_seq_act_mul": (_I, [_P, _I, _P, _I, _I, _I, _P]),
     "kb2_seq_side_gate": (_I, [_P, _P, _I, _L, _P, _I, _I, _I, _P, _I, _P]),
     "kb2_seq_latent_prep": (_I, [_P, _L, _I, _I, _I, _I, _I, _P, _F, _P, _I, _F, _P, _P, _P, _I, _I, _P, _P, _I, _P, _L, _P]),
-    "kb2_seq_latent_window_attn": (_I, [_P, _P, _L, _I, _I, _I, _I, _I, _P, _P, _I, _P, _P, _P, _I, _I, _P, _F, _I, _P, _P, _I, _I, _P, _P, _P]),
+    "kb2_seq_latent_window_attn": (_I, [_P, _P, _L, _I, _I, _I, _I, _I, _P, _P, _I, _P, _P, _P, _I, _I, _P, _F, _I, _P, _P, _I, _I, _P, _P, _P, _L, _P]),
     "kb2_seq_conv_silu": (_I, [_P, _L, _I, _I, _I, _I, _P, _P, _P, _P, _P, _P, _P]),
     "kb2_seq_delta_rule": (_I, [_P, _I, _P, _L, _I, _I, _I, _I, _I, _I, _I, _I, _I, _P, _P, _P, _F, _P, _P, _P, _P, _P, _I, _P]),
     "kb2_seq_conv": (_I, [_P, _L, _I, _I, _I, _I, _P, _P, _I, _P, _P, _P, _P, _P, _P]),
@@ -32,11 +32,11 @@ SIGNATURES = {
     "kb2_seq_head_kv_prep": (_I, [_P, _L, _I, _I, _I, _I, _I, _I, _P, _P, _P, _F, _P, _I, _P, _P, _P, _I, _I, _P, _P, _I, _I, _I, _P, _P]),
     "kb2_seq_kv_pool": (_I, [_P, _P, _P, _P, _I, _I, _I, _I, _I, _P, _P, _P, _I, _I, _P]),
     "kb2_seq_paged_attn": (_I, [_P, _L, _I, _I, _I, _I, _I, _I, _P, _P, _I, _P, _P, _P, _I, _I, _F, _I, _I, _P, _I, _P, _P, _P, _I, _F, _P, _I,
-                                _P, _P, _I, _P]),
+                                _P, _P, _I, _P, _P]),
     "kb2_seq_pool_merge": (_I, [_P, _P, _P, _P, _I, _I, _I, _P, _P, _I, _P]),
     "kb2_seq_attn_finish": (_I, [_P, _P, _P, _I, _I, _I, _I, _I, _P, _I, _F, _F, _P, _L, _P, _I, _P, _P, _I, _I, _P, _P, _I, _P]),
     "kb2_seq_glu": (_I, [_P, _I, _L, _P, _I, _L, _I, _I, _F, _F, _P, _I, _P]),
-    "kb2_seq_route": (_I, [_P, _L, _I, _I, _P, _I, _I, _I, _I, _I, _F, _P, _P, _I, _P]),
+    "kb2_seq_route": (_I, [_P, _L, _I, _I, _P, _I, _I, _I, _I, _I, _F, _P, _P, _I, _P, _P]),
     "kb2_seq_moe_tile_rows": (_I, []),
     "kb2_seq_moe_bin": (_I, [_P, _L, _I, _I, _P, _P, _P, _P, _P, _P, _L, _P, _P]),
     "kb2_seq_moe_gemm": (_I, [_P, _I, _L, _P, _I, _P, _I, _L, _L, _P, _I, _L, _I, _I, _P, _P, _I, _I, _P]),
@@ -48,6 +48,7 @@ SIGNATURES = {
     "kb2_seq_rms_rows": (_I, [_P, _L, _I, _P, _F, _P, _I, _L, _I, _P]),
     "kb2_seq_branch_merge": (_I, [_P, _P, _P, _P, _F, _F, _P, _I, _I, _P]),
     "kb2_seq_depth_mix": (_I, [_P, _L, _I, _P, _P, _P, _P, _P, _I, _I, _I, _F, _P]),
+    "kb2_seq_stream_mix": (_I, [_P, _I, _P, _P, _P, _P, _P, _P, _F, _P, _I, _I, _I, _F, _P]),
 }
 
 _lib = None
@@ -288,9 +289,13 @@ def conv(proj: torch.Tensor, C: int, taps: torch.Tensor, bias, act: bool, tail: 
     return out
 
 
+ROUTE_SCORES = {"softmax": 0, "sigmoid": 1, "top_softmax": 2}
+
+
 def route(z: torch.Tensor, correction, top: int, groups: int = 1, keep: int = 1, score: str = "softmax", renorm: bool = False,
-          out_scale: float = 1.0, group_score: str = "max", experts: int = None):
-    """Router logits z [T, >= E] fp32 -> (ids [T, top] int32, weights [T, top] fp32).  experts: E when z carries further columns.
+          out_scale: float = 1.0, group_score: str = "max", experts: int = None, bias=None):
+    """Router logits z [T, >= E] fp32 (+ bias) -> (ids [T, top] int32, weights [T, top] fp32).  experts: E when z carries further columns.
+    score: "softmax" or "sigmoid" of all logits, or "top_softmax": the largest logits are chosen, weighted by a softmax over those alone.
     group_score: "max" (a group's largest choice) or "top2" (the sum of its two largest)."""
     if z.dtype != torch.float32 or z.stride(1) != 1:
         raise ValueError("route: logits must be fp32 rows")
@@ -298,9 +303,9 @@ def route(z: torch.Tensor, correction, top: int, groups: int = 1, keep: int = 1,
     E = E if experts is None else int(experts)
     ids = torch.empty((T, top), dtype=torch.int32, device=z.device)
     w = torch.empty((T, top), dtype=torch.float32, device=z.device)
-    check(load().kb2_seq_route(z.data_ptr(), z.stride(0), T, E, _ptr(correction), {"softmax": 0, "sigmoid": 1}[score], int(groups), int(keep),
+    check(load().kb2_seq_route(z.data_ptr(), z.stride(0), T, E, _ptr(correction), ROUTE_SCORES[score], int(groups), int(keep),
                                int(top), int(renorm), float(out_scale), ids.data_ptr(), w.data_ptr(), {"max": 0, "top2": 1}[group_score],
-                               _s(z)))
+                               _ptr(bias), _s(z)))
     return ids, w
 
 
@@ -345,4 +350,19 @@ def depth_mix(stack: torch.Tensor, n: int, coef: torch.Tensor, x: torch.Tensor, 
     h = torch.empty((T, W), dtype=out_dtype, device=x.device) if norm is not None else None
     check(load().kb2_seq_depth_mix(stack.data_ptr(), stack.stride(0), n, coef.data_ptr(), x.data_ptr(), _ptr(y), _ptr(norm), _ptr(h),
                                    dt_code(out_dtype) if h is not None else 0, T, W, float(eps), _s(x)))
+    return h
+
+
+def stream_mix(xs: torch.Tensor, x0=None, y=None, mix=None, out=None, read=None, norm=None, w_shift: float = 0.0, out_dtype=torch.float32,
+               eps: float = 1e-5, want: bool = True):
+    """xs [T, n, W] fp32, n copies of the residual stream.  x0: every copy starts as x0.  y: copy t <- sum_s mix[s, t] copy_s + out[t] y.
+    Returns sum_s read[s] copy_s (read None: the plain sum), RMS-normed with w_shift + norm if norm is given, in out_dtype (None if not
+    `want`)."""
+    T, n, W = xs.shape
+    for t, shape in ((xs, xs.shape), (x0, (T, W)), (y, (T, W)), (mix, (n, n)), (out, (n,)), (read, (n,)), (norm, (W,))):
+        if t is not None and (t.dtype != torch.float32 or not t.is_contiguous() or t.shape != tuple(shape)):
+            raise ValueError("stream_mix: contiguous fp32 tensors, xs [T, n, W], x0 / y [T, W], mix [n, n], out / read [n], norm [W]")
+    h = torch.empty((T, W), dtype=out_dtype, device=xs.device) if want else None
+    check(load().kb2_seq_stream_mix(xs.data_ptr(), n, _ptr(x0), _ptr(y), _ptr(mix), _ptr(out), _ptr(read), _ptr(norm), float(w_shift), _ptr(h),
+                                    dt_code(out_dtype), T, W, float(eps), _s(xs)))
     return h
