@@ -1,4 +1,4 @@
-"""Throughput of the ragged-batch models (Vofelix, Megolorn, Gurozen, Zaronex) at layer sizes of real models, beside the framework's closest existing blocks at
+"""Throughput of the ragged-batch models (Vofelix, Megolorn, Gurozen, Zaronex, Kugalorn) at layer sizes of real models, beside the framework's closest existing blocks at
 equal size: prefill tokens/s (one prompt, whole and in portions), decode tokens/s (several live requests, one token each per step),
 and per-mixer times — the gated delta mixer against the Gated-DeltaNet block, windowed latent attention against the MLA block.
 Random weights; device timing with CUDA events after warm-up; the weights of a step exceed the L2 cache."""
@@ -576,6 +576,206 @@ def run_zaronex(args, peaks):
         blk["vofelix_decode_4_tokens_latent_attention_ms"] = round(_time(lambda: vl.forward(h4, tb4, vc_, vk_, 64), 3, 20), 4)
     except Exception as exc:       # noqa: BLE001 — the comparison is optional; the new design's numbers stand without it
         blk["comparison_unavailable"] = f"{type(exc).__name__}: {exc}"
+    out["blocks_at_equal_size"] = blk
+    out["kernels"] = kern
+    out["peaks"] = peaks
+    print(json.dumps(out))
+
+
+def kugalorn_config(width=2048, vocab=32768, window=1024, experts=64, top=6, expert_ff=1024, streams=4):
+    """Windowed attention at Gurozen's and Zaronex's attention geometry (16 heads x 128 over 2 key/value heads, window 1024), latent
+    attention at Vofelix's and Zaronex's (16 heads, 128 + 64, rank 512) over the whole context, Gurozen's number and size of experts;
+    layers 1 and 2 run twice."""
+    att = {"heads": 16, "kv_heads": 2, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": window}}
+    lat = {"heads": 16, "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": 512, "scale": 192 ** -0.5, "rot": {"base": 10000.0, "dims": 64}}
+    moe = {"kind": "moe", "router": {"experts": experts, "top": top}, "expert": {"ff": expert_ff, "limit": 7.0},
+           "shared": {"ff": 2 * expert_ff, "limit": 7.0}}
+    layers = [{"type": t, "mixer": m, "mlp": f} for t, m, f in (("attention", att, moe), ("latent_attention", lat, moe), ("attention", att, moe),
+                                                                ("latent_attention", lat, None))]
+    return {"architecture": "Kugalorn", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "streams": streams,
+            "loop": {"start": 1, "stop": 3, "times": 2}, "layers": layers}
+
+
+def _serving(model, args, prompt, out):
+    """Throughput through the scheduler: a prompt whole and in portions, decoding of four live requests, and generation end to end."""
+    from . import seqops as ops
+    from .scheduler import Scheduler
+    tokens, ctx = len(prompt), 2048
+    launches0 = ops.total_launches()
+
+    def prefill(portion):
+        s = Scheduler(model, max_tokens=tokens + 64, max_requests=4)
+        at = 0
+        while at < tokens:
+            n = min(portion, tokens - at)
+            lg = s.step([("p", prompt[at:at + n], [n - 1] if at + n == tokens else [])])
+            at += n
+        s.finish("p")
+        return lg
+    ms = _time(lambda: prefill(tokens), args.warmup, args.steps)
+    out.update(value=round(tokens / ms * 1e3, 1), ms_per_step=round(ms, 3))
+    ms_p = _time(lambda: prefill(512), 1, max(1, args.steps // 2))
+    out["prefill_portions_512"] = {"tokens_per_s": round(tokens / ms_p * 1e3, 1), "ms": round(ms_p, 3)}
+
+    s = Scheduler(model, max_tokens=4 * (ctx + 256), max_requests=4, cuda_graphs=not getattr(args, 'no_graph', False))
+    for r in range(4):
+        s.step([(r, prompt[:ctx], [])])
+    nxt = [[1], [2], [3], [4]]
+    ms_d = _time(lambda: s.step([(r, nxt[r], [0]) for r in range(4)]), args.warmup, 16)
+    out["decode"] = {"live_requests": 4, "context": ctx, "tokens_per_s": round(4 / ms_d * 1e3, 1), "ms_per_step": round(ms_d, 3),
+                     "cuda_graph": bool(s.cuda_graphs and any(v not in (None, False) for v in s._graphs.values()))}
+    out["gpu_launches"] = ops.total_launches() - launches0
+
+    s = Scheduler(model, max_tokens=tokens + 256, max_requests=4)
+    s.generate([prompt], max_new_tokens=8, step_tokens=tokens)
+    t0, t1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    torch.cuda.synchronize()
+    h2d0, steps0 = s.h2d_bytes, s.steps_run
+    t0.record()
+    s.generate([prompt], max_new_tokens=8, step_tokens=tokens)
+    t1.record()
+    torch.cuda.synchronize()
+    out["e2e"] = {"value": round((tokens + 8) / t0.elapsed_time(t1) * 1e3, 1), "unit": "tokens/s (prompt + 8 generated, Scheduler.generate)",
+                  "h2d_bytes_per_step": (s.h2d_bytes - h2d0) // max(s.steps_run - steps0, 1), "d2h_bytes_per_step": 8}
+
+
+def run_kugalorn(args, peaks):
+    from . import capi, seqops as ops
+    from .build import build, build_seq
+    build_seq()
+    build()                                          # the tcgen05 GEMM and attention core serve long bfloat16 steps
+    from .attention import HeadKVCache
+    from .kugalorn import KugalornConfig, KugalornModel
+    dev = torch.device("cuda", 0)
+    tokens = args.tokens or 4096
+    raw = kugalorn_config()
+    cfg = KugalornConfig.from_dict(raw)
+    model = KugalornModel.random(cfg, seed=0, dtype=torch.bfloat16, device=0)
+    g = torch.Generator().manual_seed(0)
+    prompt = torch.randint(0, cfg.vocab, (tokens,), generator=g).tolist()
+    out = {"metric": "kugalorn_prefill_tokens_per_s", "unit": "tokens/s", "n_gpus": 1, "steps": args.steps, "warmup": args.warmup,
+           "higher_is_better": True, "dtype": "bf16", "data": "synthetic (random weights and token ids)", "vs_baseline": None,
+           "config": {"model": "kugalorn width 2048, 4 stream copies: 4 layers (attention 16 heads x 128 / 2 kv heads, window 1024, distance "
+                               "penalty; latent attention 16 heads 128+64 / rank 512, gate per head), layers 1..2 run twice = 6 layer runs; 64 "
+                               "clamped-swish experts, top 6, expert ff 1024, shared ff 2048 (last layer without)", "prompt_tokens": tokens,
+                      "l2": "weights of one step (about 2.8 GB) exceed L2"}}
+    _serving(model, args, prompt, out)
+
+    # ---- per-block times, prefill and decode, beside the closest blocks of the other designs at equal size
+    blk, W, ctx = {}, cfg.width, 2048
+    h = (torch.randn(tokens, W, generator=g) * 0.5).to(torch.bfloat16).to(dev)
+    h4 = h[:4].contiguous()
+    pages = list(range((tokens + 63) // 64))
+    tb = ops.StepTables([(prompt, 0, 0, pages)], dev)
+    tb4 = ops.StepTables([([1], ctx, r, list(range(r * 40, r * 40 + 33))) for r in range(4)], dev)
+    model.make_caches(max(tokens, 4 * 40 * 64) + 64, 4)
+    kvc = model.kv_cache
+    for t in kvc.k + kvc.v:                          # finite, ordinary contents: what decode reads at once
+        t.copy_((torch.randn(t.shape, device=dev) * 0.5).to(t.dtype))
+    att, lat, moe = model.layers[0]["mixer"], model.layers[1]["mixer"], model.layers[0]["mlp"]
+
+    def both(name, fn_of):                           # fn_of(h, tables) -> callable
+        blk[name + "_ms"] = round(_time(fn_of(h, tb), 2, 5), 3)
+        blk["decode_4_tokens_" + name + "_ms"] = round(_time(fn_of(h4, tb4), 3, 20), 4)
+    both("windowed_attention_block", lambda hh, t: (lambda: att.forward(hh, t, *kvc.get_layer_caches(0), 64)))
+    both("latent_attention_block", lambda hh, t: (lambda: lat.forward(hh, t, *kvc.get_layer_caches(1), 64)))
+    both("routed_experts_block", lambda hh, t: (lambda: moe.forward(hh)))
+    try:                                             # the closest blocks of the other designs, built at this design's sizes
+        from .gurozen import GurozenConfig, GurozenModel
+        from .megolorn import MegolornConfig, MegolornModel
+        from .vofelix import VofelixConfig, VofelixModel
+        from .zaronex import ZaronexConfig, ZaronexModel
+        zraw = zaronex_config()
+        zraw["layers"] = [zraw["layers"][2]]
+        zm = ZaronexModel.random(ZaronexConfig.from_dict(zraw), seed=0, dtype=torch.bfloat16, device=0)
+        za = zm.layers[0]["mixer"].left
+        both("zaronex_rotated_value_attention_block", lambda hh, t: (lambda: za.forward(hh, t, *kvc.get_layer_caches(0), 64)))
+        graw = gurozen_config()
+        graw["layers"] = [dict(graw["layers"][0], mlp=graw["layers"][1]["mlp"])]
+        graw["loop"] = {"start": 0, "stop": 0, "times": 0}
+        gm = GurozenModel.random(GurozenConfig.from_dict(graw), seed=0, dtype=torch.bfloat16, device=0)
+        both("gurozen_routed_experts_block", lambda hh, t: (lambda: gm.layers[0]["mlp"].forward(hh)))
+        mraw = megolorn_config(experts=64, identity=0)
+        mraw["layers"] = [dict(mraw["layers"][0], mlp=mraw["layers"][1]["mlp"])]
+        mm = MegolornModel.random(MegolornConfig.from_dict(mraw), seed=0, dtype=torch.bfloat16, device=0)
+        both("megolorn_routed_experts_block", lambda hh, t: (lambda: mm.layers[0]["mlp"].forward(hh)))
+        vraw, _, vlat = bench_config()
+        vraw["layers"] = [_layer("latent_attention", dict(vlat, mask={"size": 1 << 20}))]      # the window open, like this design's
+        vraw["loop"] = {"start": 0, "stop": 0, "times": 1}
+        vm = VofelixModel.random(VofelixConfig.from_dict(vraw), seed=0, dtype=torch.bfloat16, device=0)
+        vl = vm.layers[0]["mixer"]
+        both("vofelix_latent_attention_block_open_window", lambda hh, t: (lambda: vl.forward(hh, t, *kvc.get_layer_caches(1), 64)))
+    except Exception as exc:       # noqa: BLE001 — the comparison is optional; the new design's numbers stand without it
+        blk["comparison_unavailable"] = f"{type(exc).__name__}: {exc}"
+
+    # ---- the new kernels alone, each beside the like kernel: time, algorithmic bytes and flops, fractions of the measured peaks
+    kern, lib, core = {}, ops.load(), capi.load()
+    cs = torch.cuda.current_stream(dev).cuda_stream
+
+    def kernel(name, fn, nbytes, flops=0.0, reps=(3, 20)):
+        ms_k = _time(fn, *reps)
+        e = {"ms": round(ms_k, 4), "GB_per_s": round(nbytes / ms_k / 1e6, 1), "of_measured_hbm": round(nbytes / ms_k / 1e6 / peaks["hbm_gbs"], 3)}
+        if flops:
+            e.update(TFLOP_per_s=round(flops / ms_k / 1e9, 2), of_measured_bf16=round(flops / ms_k / 1e9 / peaks["bf16_tflops"], 3))
+        kern[name] = e
+    n = cfg.streams
+    rnd = lambda *s: torch.randn(*s, device=dev)
+    for label, T_ in (("prefill_4096", tokens), ("decode_4", 4)):
+        xs, y, x, nw = rnd(T_, n, W), rnd(T_, W), rnd(T_, W), rnd(W)
+        mix, o_, r_ = rnd(n, n) * 0.3, rnd(n), rnd(n)
+        kernel(f"stream_mix_{n}_copies_{label}", lambda: ops.stream_mix(xs, y=y, mix=mix, out=o_, read=r_, norm=nw, w_shift=1.0,
+                                                                         out_dtype=torch.bfloat16), T_ * W * (8 * n + 4 + 2))
+        stack, coef = rnd(n + 1, T_, W), rnd(n + 1)
+        hb = torch.empty(T_, W, dtype=torch.bfloat16, device=dev)
+        kernel(f"depth_mix_{n + 1}_results_{label} (like kernel: Zaronex)",
+               lambda: ops.check(lib.kb2_seq_depth_mix(stack.data_ptr(), stack.stride(0), n + 1, coef.data_ptr(), x.data_ptr(), y.data_ptr(),
+                                                       nw.data_ptr(), hb.data_ptr(), 1, T_, W, 1e-6, cs)), T_ * W * (4 * n + 4 + 4 + 4 + 4 + 2))
+        kernel(f"residual_scale_rms_{label} (like kernel: Gurozen)",
+               lambda: ops.residual_scale_rms(x, y, 1.0, norm=nw, out_dtype=torch.bfloat16), T_ * W * 14)
+        z, rb = rnd(T_, 64), rnd(64)
+        kernel(f"route_top_softmax_{label}", lambda: ops.route(z, None, 6, score="top_softmax", bias=rb), T_ * (64 * 4 + 48))
+        kernel(f"route_softmax_{label} (like kernel: Megolorn)", lambda: ops.route(z, None, 6), T_ * (64 * 4 + 48))
+    H, G, d, win = att.H, att.G, att.d, att.window
+    bf = lambda *s: rnd(*s).to(torch.bfloat16)
+    q, k, v = bf(tokens, H * d), bf(tokens, G * d), bf(tokens, G * d)
+    o = torch.empty(tokens, H * d, device=dev)
+    pairs = sum(min(i + 1, win) for i in range(tokens))
+    fl, by = 4.0 * pairs * H * d, tokens * (H * d * 2 + 2 * G * d * 2 + H * d * 4)
+    core_args = (q.data_ptr(), k.data_ptr(), v.data_ptr(), o.data_ptr(), tokens, 0, tokens, H, G, 1, d, d ** -0.5, 0.0, win, None, None)
+    kernel("attention_core_distance_penalty_prefill_4096", lambda: capi.check(core.kb2_fmha_maps_slopes(*core_args, att.map_slopes.data_ptr(), 0, cs)), by, fl)
+    kernel("attention_core_prefill_4096 (like kernel: Zaronex, window without penalty)", lambda: capi.check(core.kb2_fmha_maps_sink(*core_args, 0, cs)), by, fl)
+    Hl = lat.H
+    ql, kvu, kpe = bf(tokens, Hl * 192), bf(tokens, Hl * 256), bf(tokens, 64)
+    ol, gate = torch.empty(tokens, Hl * 128, dtype=torch.bfloat16, device=dev), rnd(tokens, Hl)
+    fl, by = 2.0 * (tokens * (tokens + 1) // 2) * Hl * (192 + 128), tokens * (Hl * (192 + 256 + 128) + 64) * 2
+    lat_args = (ql.data_ptr(), kvu.data_ptr(), kpe.data_ptr(), ol.data_ptr(), tokens, 0, tokens, Hl, 192 ** -0.5, 1 << 30, None)
+    kernel("latent_core_gate_per_head_prefill_4096", lambda: capi.check(core.kb2_fmha_latent_gated(*lat_args, gate.data_ptr(), Hl, 0, cs)), by, fl)
+    kernel("latent_core_prefill_4096 (like kernel: Vofelix)", lambda: capi.check(core.kb2_fmha_latent(*lat_args, 0, cs)), by, fl)
+    # decoding: 4 tokens at 2048 of context over the pages, key range cut into pieces as the blocks do
+    kc, vc = kvc.get_layer_caches(0)
+    proj, nsp = rnd(4, (H + 2 * G) * d), max(1, min(296 // (4 * G), (win + 31) // 32, 64))
+    pa, pm, oo = rnd(4 * H, nsp, d), rnd(4 * H, nsp, 2), rnd(4, H, d)
+
+    def decode_attn(slopes):
+        ops.check(lib.kb2_seq_paged_attn(proj.data_ptr(), proj.stride(0), 4, H, G, 1, d, d, kc.data_ptr(), vc.data_ptr(), 1, tb4.positions.data_ptr(),
+                                         tb4.seq_of.data_ptr(), tb4.pages.data_ptr(), tb4.max_pages, 64, d ** -0.5, 0, win, oo.data_ptr(), nsp,
+                                         pa.data_ptr(), pm.data_ptr(), None, 0, 0.0, None, 0, None, None, 0, slopes, cs))
+    by = 4 * win * 2 * G * d * 2
+    kernel("paged_attn_distance_penalty_decode_4", lambda: decode_attn(att.slopes.data_ptr()), by)
+    kernel("paged_attn_decode_4 (like kernel: Zaronex)", lambda: decode_attn(None), by)
+    ck, kr = kvc.get_layer_caches(1)
+    ql4, qa = rnd(4, Hl * 192 + 576 + Hl), rnd(4, Hl, 512)
+    nsp2 = max(1, min(296 // (4 * ((Hl + 7) // 8)), (ctx + 32) // 32, 64))
+    la, lm, lo = rnd(4, nsp2, Hl, 512), rnd(4, nsp2, Hl, 2), rnd(4, Hl, 512)
+
+    def decode_latent(gt):
+        ops.check(lib.kb2_seq_latent_window_attn(qa.data_ptr(), ql4.data_ptr(), ql4.stride(0), 4, Hl, 128, 64, 512, ck.data_ptr(), kr.data_ptr(), 1,
+                                                 tb4.positions.data_ptr(), tb4.seq_of.data_ptr(), tb4.pages.data_ptr(), tb4.max_pages, 64, None,
+                                                 192 ** -0.5, 1 << 30, lo.data_ptr(), None, 0, nsp2, la.data_ptr(), lm.data_ptr(), gt,
+                                                 ql4.stride(0), cs))
+    by = 4 * (ctx + 1) * 576 * 2
+    kernel("latent_attn_gate_per_head_decode_4", lambda: decode_latent(ql4[:, Hl * 192 + 576:].data_ptr()), by)
+    kernel("latent_attn_decode_4 (like kernel: Vofelix)", lambda: decode_latent(None), by)
     out["blocks_at_equal_size"] = blk
     out["kernels"] = kern
     out["peaks"] = peaks
