@@ -716,7 +716,7 @@ def run_kugalorn(args, peaks):
         ms_k = _time(fn, *reps)
         e = {"ms": round(ms_k, 4), "GB_per_s": round(nbytes / ms_k / 1e6, 1), "of_measured_hbm": round(nbytes / ms_k / 1e6 / peaks["hbm_gbs"], 3)}
         if flops:
-            e.update(TFLOP_per_s=round(flops / ms_k / 1e9, 2), of_measured_bf16=round(flops / ms_k / 1e9 / peaks["bf16_tflops"], 3))
+            e.update(TFLOP_per_s=round(flops / ms_k / 1e9, 2), of_measured_bf16=round(flops / ms_k / 1e9 / peaks["tf_burst"], 3))
         kern[name] = e
     n = cfg.streams
     rnd = lambda *s: torch.randn(*s, device=dev)

@@ -61,6 +61,12 @@ __device__ __forceinline__ void unpack8(const uint4& v, float* f) {
     f[2 * i + 1] = t.y;
   }
 }
+// streamed once: keep the weights out of L1 so that the few activation rows every warp re-reads stay there
+__device__ __forceinline__ uint4 ld_stream16(const void* p) {
+  uint4 v;
+  asm volatile("ld.global.nc.L1::no_allocate.v4.u32 {%0, %1, %2, %3}, [%4];" : "=r"(v.x), "=r"(v.y), "=r"(v.z), "=r"(v.w) : "l"(p));
+  return v;
+}
 __device__ __forceinline__ float gelu_tanh(float z) {
   return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
 }

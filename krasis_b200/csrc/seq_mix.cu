@@ -319,8 +319,10 @@ __global__ void __launch_bounds__(kPAThreads) paged_attn_kernel(
 }
 
 // A warp per (token, head): o = sum_m coef[m] a_m (a_m merged from its key pieces when nsplit > 1), o / rms(o) * post_scale if
-// unit_norm, times sigmoid(gate[t, h]) if gates are given.  dv <= 32 * kFinAcc.
-constexpr int kFinAcc = 16;
+// unit_norm, times sigmoid(gate[t, h]) if gates are given.  NA: columns per lane,
+// dv <= 32 NA.
+constexpr int kFinAcc = 16;               // the most columns per lane
+template <int NA>
 __global__ void __launch_bounds__(256) attn_finish_kernel(const float* __restrict__ a, const float* __restrict__ part_acc,
                                                           const float* __restrict__ part_ml, int nsplit, long long T, int H, int M, int dv,
                                                           const float* __restrict__ coef, int unit_norm, float eps, float post_scale,
@@ -328,7 +330,7 @@ __global__ void __launch_bounds__(256) attn_finish_kernel(const float* __restric
                                                           int dt_out, const int* __restrict__ seq_of, const int* __restrict__ cu,
                                                           int skip_from, int gate_wide, const int* __restrict__ positions,
                                                           const double* __restrict__ vfreq, int rot_half) {
-  __shared__ float turn_buf[8][32 * kFinAcc];
+  __shared__ float turn_buf[8][32 * NA];
   const long long w = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
   const int lane = threadIdx.x & 31;
   if (w >= T * H) return;
@@ -338,9 +340,9 @@ __global__ void __launch_bounds__(256) attn_finish_kernel(const float* __restric
     const int sq = seq_of[t];
     if (cu[sq + 1] - cu[sq] >= skip_from) return;
   }
-  float o[kFinAcc];
+  float o[NA];
 #pragma unroll
-  for (int i = 0; i < kFinAcc; ++i) o[i] = 0.f;
+  for (int i = 0; i < NA; ++i) o[i] = 0.f;
   for (int m = 0; m < M; ++m) {
     const long long row = w * M + m;
     const float cm = coef ? coef[m] : 1.f;
@@ -366,7 +368,7 @@ __global__ void __launch_bounds__(256) attn_finish_kernel(const float* __restric
         for (int k = 0; k < nz; ++k) {
           const float wz = __shfl_sync(0xffffffffu, wl, k);
 #pragma unroll
-          for (int i = 0; i < kFinAcc; ++i) {
+          for (int i = 0; i < NA; ++i) {
             const int c = lane + 32 * i;
             if (c < dv) o[i] = fmaf(wz, part_acc[(row * nsplit + z0 + k) * dv + c], o[i]);
           }
@@ -374,7 +376,7 @@ __global__ void __launch_bounds__(256) attn_finish_kernel(const float* __restric
       }
     } else {
 #pragma unroll
-      for (int i = 0; i < kFinAcc; ++i) {
+      for (int i = 0; i < NA; ++i) {
         const int c = lane + 32 * i;
         if (c < dv) o[i] = fmaf(cm, a[row * dv + c], o[i]);
       }
@@ -384,21 +386,21 @@ __global__ void __launch_bounds__(256) attn_finish_kernel(const float* __restric
   if (unit_norm) {
     float ss = 0.f;
 #pragma unroll
-    for (int i = 0; i < kFinAcc; ++i) ss += o[i] * o[i];
+    for (int i = 0; i < NA; ++i) ss += o[i] * o[i];
     ss = warp_sum(ss);
     f = post_scale / sqrtf(ss / (float)dv + eps);
   }
   if (vfreq != nullptr) {       // values were cached rotated by their positions: turn the sum back by the query's position
     float* tb = turn_buf[threadIdx.x >> 5];
 #pragma unroll
-    for (int i = 0; i < kFinAcc; ++i) {
+    for (int i = 0; i < NA; ++i) {
       const int c = lane + 32 * i;
       if (c < dv) tb[c] = o[i];
     }
     __syncwarp();
     const int vh = dv >> 1, pos = positions[t];
 #pragma unroll
-    for (int i = 0; i < kFinAcc; ++i) {
+    for (int i = 0; i < NA; ++i) {
       const int c = lane + 32 * i;
       if (c < dv) {
         const int j = rot_half ? (c < vh ? c : c - vh) : c >> 1;
@@ -412,7 +414,7 @@ __global__ void __launch_bounds__(256) attn_finish_kernel(const float* __restric
   }
   if (gate != nullptr && !gate_wide) f *= 1.f / (1.f + expf(-gate[t * ldg + h]));
 #pragma unroll
-  for (int i = 0; i < kFinAcc; ++i) {
+  for (int i = 0; i < NA; ++i) {
     const int c = lane + 32 * i;
     if (c < dv) {
       float v = o[i] * f;
@@ -709,7 +711,17 @@ __global__ void __launch_bounds__(256) moe_gemv_kernel(const TA* __restrict__ A,
   const TA* a = A + (long long)(slot / div) * lda;
   const TB* b = B + (long long)e * sB + (long long)n * ldb;
   float acc = 0.f;
-  if (sizeof(TB) == 2 && (K & 7) == 0 && (ldb & 7) == 0 && (sB & 7) == 0 && !((uintptr_t)B & 15)) {
+  if (sizeof(TB) == 2 && sizeof(TA) == 2 && (K & 7) == 0 && (ldb & 7) == 0 && (sB & 7) == 0 && (lda & 7) == 0 && !((uintptr_t)B & 15) &&
+      !((uintptr_t)A & 15)) {
+#pragma unroll 4
+    for (int k = lane * 8; k < K; k += 256) {          // 16-byte loads of both rows, those of four pieces in flight together
+      float wv[8], av[8];
+      unpack8(ld_stream16(b + k), wv);
+      unpack8(*reinterpret_cast<const uint4*>(a + k), av);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) acc = fmaf(av[i], wv[i], acc);
+    }
+  } else if (sizeof(TB) == 2 && (K & 7) == 0 && (ldb & 7) == 0 && (sB & 7) == 0 && !((uintptr_t)B & 15)) {
     for (int k = lane * 8; k < K; k += 256) {
       float wv[8];
       unpack8(*reinterpret_cast<const uint4*>(b + k), wv);
@@ -857,9 +869,14 @@ KB2SEQ_API int kb2_seq_attn_finish(const float* a, const float* part_acc, const 
     return failf(KB2SEQ_ERR_VALUE, "attn_finish: bad argument");
   if (dv > 32 * kFinAcc) return failf(KB2SEQ_ERR_VALUE, "attn_finish: value size %d > %d", dv, 32 * kFinAcc);
   const long long nwarps = (long long)T * H;
-  attn_finish_kernel<<<(unsigned)((nwarps + 7) / 8), 256, 0, (cudaStream_t)stream>>>(a, part_acc, part_ml, nsplit, T, H, M, dv, coef, unit_norm,
-                                                                                      eps, post_scale, gate, ldg, out, dt_out, seq_of, cu,
-                                                                                      skip_from, gate_wide, positions, vfreq, rot_half);
+#define KB2_FIN(NAV)                                                                                                                        \
+  attn_finish_kernel<NAV><<<(unsigned)((nwarps + 7) / 8), 256, 0, (cudaStream_t)stream>>>(a, part_acc, part_ml, nsplit, T, H, M, dv, coef, unit_norm, \
+                                                                                         eps, post_scale, gate, ldg, out, dt_out, seq_of, cu, skip_from, \
+                                                                                         gate_wide, positions, vfreq, rot_half)
+  if (dv <= 128) KB2_FIN(4);
+  else if (dv <= 256) KB2_FIN(8);
+  else KB2_FIN(16);
+#undef KB2_FIN
   SEQ_LAUNCHED();
   return KB2SEQ_OK;
 }

@@ -118,12 +118,6 @@ __global__ void __launch_bounds__(256) gemv_nt_kernel(const TA* __restrict__ A, 
   }
 }
 
-// streamed once: keep the weights out of L1 so that the few activation rows every warp re-reads stay there
-__device__ __forceinline__ uint4 ld_stream16(const void* p) {
-  uint4 v;
-  asm volatile("ld.global.nc.L1::no_allocate.v4.u32 {%0, %1, %2, %3}, [%4];" : "=r"(v.x), "=r"(v.y), "=r"(v.z), "=r"(v.w) : "l"(p));
-  return v;
-}
 template <typename TA> __device__ __forceinline__ void load8(const TA* p, float* f);
 template <> __device__ __forceinline__ void load8<float>(const float* p, float* f) {
   const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
@@ -424,30 +418,42 @@ __global__ void __launch_bounds__(128) latent_prep_kernel(float* __restrict__ pr
 // Absorbed form: score(t, h, j) = (q_abs[t,h] . c_j + q_rot[t,h] . kr_j) * scale over the keys j of the token's sequence with
 // 0 <= pos - j < window; the softmax denominator also holds exp(sink_h) (a key with no value: running max starts at the sink,
 // running sum at 1).  Output: sum_j p_j c_j (the value up-projection follows as a per-head GEMM).
-// One block per (token, group of HG heads); keys in tiles of KT, shared by the heads of the group.
+// One block per (token, group of HG heads, piece of the key range); keys in tiles of 32, in shared memory as fp32 rows whose pitch is an
+// odd number of 16-byte units, so that a lane per key reads 16 bytes without bank conflicts.
+//   scores    every warp takes an eighth of the dimensions for all HG heads: one 16-byte read of a key row serves HG dot products, whose
+//             pieces meet in shared memory
+//   values    a thread owns NC columns for all HG heads: one read of a latent element serves HG sums
 // gate [T, ldg] (may be null): head h's output is multiplied by sigmoid(gate[t, h]); it commutes with the value up-projection.
-constexpr int kAttnThreads = 256, kAttnAcc = 16;
+constexpr int kAttnThreads = 256, kAttnAcc = 16, kAttnKT = 32, kAttnWarps = kAttnThreads / 32;
 __device__ __forceinline__ float head_gate(const float* __restrict__ gate, long long ldg, long long t, int h) {
   return gate != nullptr ? 1.f / (1.f + expf(-gate[t * ldg + h])) : 1.f;
 }
-__global__ void __launch_bounds__(kAttnThreads) latent_window_attn_kernel(
-    const float* __restrict__ q_abs, const float* __restrict__ proj, long long ldp, int H, int HG, int dn, int dr, int r,
+__host__ __device__ inline int attn_q_pitch(int D) { return (D + 3) / 4 * 4; }
+__host__ __device__ inline int attn_k_pitch(int D) { return attn_q_pitch(D) / 4 % 2 ? attn_q_pitch(D) : attn_q_pitch(D) + 4; }
+__host__ __device__ inline size_t attn_smem_floats(int HG, int D) {
+  return 2 * kAttnKT + (size_t)HG * attn_q_pitch(D) + (size_t)kAttnKT * attn_k_pitch(D) + (size_t)kAttnWarps * HG * kAttnKT + (size_t)kAttnKT * HG + 3 * HG;
+}
+template <int HG, int NC>
+__global__ void __launch_bounds__(kAttnThreads, 2) latent_window_attn_kernel(
+    const float* __restrict__ q_abs, const float* __restrict__ proj, long long ldp, int H, int dn, int dr, int r,
     const void* __restrict__ ckv, const void* __restrict__ kr, int dt_cache, const int* __restrict__ positions,
     const int* __restrict__ seq_of, const int* __restrict__ pages, int max_pages, int page_size, const float* __restrict__ sinks,
-    float scale, int window, int KT, float* __restrict__ out, const int* __restrict__ cu, int skip_from, int nsplit,
+    float scale, int window, float* __restrict__ out, const int* __restrict__ cu, int skip_from, int nsplit,
     float* __restrict__ part_acc, float* __restrict__ part_ml, const float* __restrict__ gate, long long ldg) {
+  static_assert(HG <= kAttnWarps, "a warp per head runs the softmax");
+  constexpr int KT = kAttnKT;
   extern __shared__ __align__(16) float sm[];
   if (cu != nullptr) {                    // sequences whose portion has skip_from tokens or more are served by another kernel
     const int sq = seq_of[blockIdx.x];
     if (cu[sq + 1] - cu[sq] >= skip_from) return;
   }
-  const int D = r + dr, DP = D + 1;
+  const int D = r + dr, QP = attn_q_pitch(D), DP = attn_k_pitch(D), n4 = QP >> 2;
   long long* krow = (long long*)sm;       // [KT] cache rows of the tile's keys
-  float* qs = sm + 2 * KT;                // [HG][D]
-  float* kt = qs + HG * D;                // [KT][DP]
-  float* pr = kt + KT * DP;               // [HG][KT]
-  float* sp = pr + HG * KT;               // [warps][KT] partial scores: a head's dot product is cut into warps / HG pieces
-  float* m_run = sp + (kAttnThreads / 32) * KT;   // [HG]
+  float* qs = sm + 2 * KT;                // [HG][QP], zeros beyond the head's D numbers and beyond the last head
+  float* kt = qs + HG * QP;               // [KT][DP]
+  float* sp = kt + KT * DP;               // [warps][HG][KT] pieces of the scores
+  float* pr = sp + kAttnWarps * HG * KT;  // [KT][HG] weights
+  float* m_run = pr + KT * HG;            // [HG]
   float* l_run = m_run + HG;              // [HG]
   float* alpha = l_run + HG;              // [HG]
   const long long t = blockIdx.x;
@@ -455,21 +461,29 @@ __global__ void __launch_bounds__(kAttnThreads) latent_window_attn_kernel(
   const int nh = min(HG, H - h0);
   const int pos = positions[t], seq = seq_of[t];
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-  for (int i = tid; i < nh * D; i += kAttnThreads) {
-    const int hh = i / D, d = i - hh * D;
-    qs[i] = d < r ? q_abs[(t * H + h0 + hh) * r + d] : proj[t * ldp + (long long)(h0 + hh) * (dn + dr) + dn + (d - r)];
+  for (int i = tid; i < HG * QP; i += kAttnThreads) {
+    const int hh = i / QP, d = i - hh * QP;
+    float v = 0.f;
+    if (hh < nh && d < D) v = d < r ? q_abs[(t * H + h0 + hh) * r + d] : proj[t * ldp + (long long)(h0 + hh) * (dn + dr) + dn + (d - r)];
+    qs[i] = v;
+  }
+  for (int i = tid; i < KT * (DP - D); i += kAttnThreads) {      // the rows' padding stays zero: tiles write D numbers per row only
+    const int k = i / (DP - D);
+    kt[k * DP + D + i - k * (DP - D)] = 0.f;
   }
   // nsplit > 1: block z takes the z-th piece of the token's key range and leaves an unnormalised partial result (running max, sum,
   // weighted latents) for latent_attn_combine_kernel; the sink belongs to piece 0
   const int z = blockIdx.z;
-  if (tid < nh) {
-    const bool sk = z == 0 && sinks != nullptr;       // no sinks: an ordinary softmax over the keys
+  if (tid < HG) {
+    const bool sk = z == 0 && sinks != nullptr && tid < nh;       // no sinks: an ordinary softmax over the keys
     m_run[tid] = sk ? sinks[h0 + tid] : -INFINITY;
     l_run[tid] = sk ? 1.f : 0.f;
   }
-  float acc[kAttnAcc];
+  float acc[NC][HG];
 #pragma unroll
-  for (int a = 0; a < kAttnAcc; ++a) acc[a] = 0.f;
+  for (int c = 0; c < NC; ++c)
+#pragma unroll
+    for (int hh = 0; hh < HG; ++hh) acc[c][hh] = 0.f;
   const int j_lo = max(0, pos - window + 1);
   int j_begin = j_lo, j_end = pos;
   if (nsplit > 1) {
@@ -477,6 +491,7 @@ __global__ void __launch_bounds__(kAttnThreads) latent_window_attn_kernel(
     j_begin = j_lo + z * piece;
     j_end = min(pos, j_begin + piece - 1);
   }
+  const int seg = (n4 + kAttnWarps - 1) / kAttnWarps, u_lo = min(n4, warp * seg), u_hi = min(n4, u_lo + seg);
   for (int j0 = j_begin; j0 <= j_end; j0 += KT) {
     const int nk = min(KT, j_end - j0 + 1);
     __syncthreads();
@@ -492,8 +507,8 @@ __global__ void __launch_bounds__(kAttnThreads) latent_window_attn_kernel(
         const bf16* src = d < r ? (const bf16*)ckv + krow[k] * r + d : (const bf16*)kr + krow[k] * dr + (d - r);
         float f[8];
         unpack8(*reinterpret_cast<const uint4*>(src), f);
-#pragma unroll
-        for (int e = 0; e < 8; ++e) kt[k * DP + d + e] = f[e];
+        *reinterpret_cast<float4*>(kt + k * DP + d) = make_float4(f[0], f[1], f[2], f[3]);
+        *reinterpret_cast<float4*>(kt + k * DP + d + 4) = make_float4(f[4], f[5], f[6], f[7]);
       }
     } else {
       for (int i = tid; i < nk * D; i += kAttnThreads) {
@@ -502,72 +517,101 @@ __global__ void __launch_bounds__(kAttnThreads) latent_window_attn_kernel(
       }
     }
     __syncthreads();
-    // scores: warp w takes piece w / HG of head w % HG, a lane per key (HG is a power of two <= 8, KT == 32)
+    // scores: a lane per key, a piece of the dimensions per warp, all heads of the group
     {
-      const int P = (kAttnThreads / 32) / HG, part = warp / HG, hw = warp % HG;
-      const int dseg = (D + P - 1) / P, d_lo = part * dseg, d_hi = min(D, d_lo + dseg);
-      float dot = 0.f;
-      if (hw < nh && lane < nk) {
-        const float* qh = qs + hw * D;
-        const float* kk = kt + lane * DP;
-        for (int d = d_lo; d < d_hi; ++d) dot = fmaf(qh[d], kk[d], dot);
+      float s[HG];
+#pragma unroll
+      for (int hh = 0; hh < HG; ++hh) s[hh] = 0.f;
+      if (lane < nk) {
+        const float4* kk = reinterpret_cast<const float4*>(kt + lane * DP);
+        const float4* qq = reinterpret_cast<const float4*>(qs);
+        for (int u = u_lo; u < u_hi; ++u) {
+          const float4 kv = kk[u];
+#pragma unroll
+          for (int hh = 0; hh < HG; ++hh) {
+            const float4 qv = qq[hh * n4 + u];
+            s[hh] = fmaf(qv.x, kv.x, s[hh]);
+            s[hh] = fmaf(qv.y, kv.y, s[hh]);
+            s[hh] = fmaf(qv.z, kv.z, s[hh]);
+            s[hh] = fmaf(qv.w, kv.w, s[hh]);
+          }
+        }
       }
-      sp[warp * KT + lane] = dot;
+#pragma unroll
+      for (int hh = 0; hh < HG; ++hh) sp[(warp * HG + hh) * KT + lane] = s[hh];
     }
     __syncthreads();
-    // running softmax: warp hh < nh
-    for (int hh = warp; hh < nh; hh += kAttnThreads / 32) {
-      const float m_old = m_run[hh];
-      float m_new = m_old;
-      {
-        const int P = (kAttnThreads / 32) / HG;
+    // running softmax: warp hh serves head hh
+    if (warp < HG) {
+      float p = 0.f;
+      if (warp < nh) {
+        const float m_old = m_run[warp];
         float sc = -INFINITY;
         if (lane < nk) {
           float dot = 0.f;
-          for (int pp = 0; pp < P; ++pp) dot += sp[(pp * HG + hh) * KT + lane];
+#pragma unroll
+          for (int w = 0; w < kAttnWarps; ++w) dot += sp[(w * HG + warp) * KT + lane];
           sc = dot * scale;
         }
-        pr[hh * KT + lane] = sc;
-        m_new = fmaxf(m_new, warp_max(sc));
-      }
-      float lsum = 0.f;
-      for (int kb = 0; kb < nk; kb += 32) {
-        const int k = kb + lane;
-        float p = 0.f;
-        if (k < nk) {
-          p = expf(pr[hh * KT + k] - m_new);
-          pr[hh * KT + k] = p;
+        const float m_new = fmaxf(m_old, warp_max(sc));
+        if (lane < nk) p = expf(sc - m_new);
+        const float lsum = warp_sum(p);
+        if (lane == 0) {
+          const float al = m_old == -INFINITY ? 0.f : expf(m_old - m_new);
+          alpha[warp] = al;
+          l_run[warp] = l_run[warp] * al + lsum;
+          m_run[warp] = m_new;
         }
-        lsum += warp_sum(p);
+      } else if (lane == 0) {
+        alpha[warp] = 0.f;
       }
-      if (lane == 0) {
-        const float al = m_old == -INFINITY ? 0.f : expf(m_old - m_new);
-        alpha[hh] = al;
-        l_run[hh] = l_run[hh] * al + lsum;
-        m_run[hh] = m_new;
-      }
+      pr[lane * HG + warp] = p;
     }
     __syncthreads();
+    {
 #pragma unroll
-    for (int a = 0; a < kAttnAcc; ++a) {
-      const int i = tid + a * kAttnThreads;
-      if (i < nh * r) {
-        const int hh = i / r, d = i - hh * r;
-        float v = acc[a] * alpha[hh];
-        const float* ph = pr + hh * KT;
-        for (int k = 0; k < nk; ++k) v = fmaf(ph[k], kt[k * DP + d], v);
-        acc[a] = v;
+      for (int hh = 0; hh < HG; ++hh) {
+        const float al = alpha[hh];
+#pragma unroll
+        for (int c = 0; c < NC; ++c) acc[c][hh] *= al;
+      }
+      for (int k = 0; k < nk; ++k) {
+        float p[HG];
+        if constexpr (HG % 4 == 0) {
+#pragma unroll
+          for (int q = 0; q < HG / 4; ++q) {
+            const float4 f = *reinterpret_cast<const float4*>(pr + k * HG + 4 * q);
+            p[4 * q] = f.x; p[4 * q + 1] = f.y; p[4 * q + 2] = f.z; p[4 * q + 3] = f.w;
+          }
+        } else {
+#pragma unroll
+          for (int hh = 0; hh < HG; ++hh) p[hh] = pr[k * HG + hh];
+        }
+#pragma unroll
+        for (int c = 0; c < NC; ++c) {
+          const int d = tid + c * kAttnThreads;
+          if (d < r) {
+            const float v = kt[k * DP + d];
+#pragma unroll
+            for (int hh = 0; hh < HG; ++hh) acc[c][hh] = fmaf(p[hh], v, acc[c][hh]);
+          }
+        }
       }
     }
   }
   __syncthreads();
 #pragma unroll
-  for (int a = 0; a < kAttnAcc; ++a) {
-    const int i = tid + a * kAttnThreads;
-    if (i < nh * r) {
-      const int hh = i / r, d = i - hh * r;
-      if (nsplit > 1) part_acc[((t * nsplit + z) * H + h0 + hh) * r + d] = acc[a];
-      else out[(t * H + h0 + hh) * r + d] = acc[a] / l_run[hh] * head_gate(gate, ldg, t, h0 + hh);
+  for (int hh = 0; hh < HG; ++hh) {
+    if (hh >= nh) continue;
+    const float f = nsplit > 1 ? 1.f : head_gate(gate, ldg, t, h0 + hh);
+    const float l = l_run[hh];
+#pragma unroll
+    for (int c = 0; c < NC; ++c) {
+      const int d = tid + c * kAttnThreads;
+      if (d < r) {
+        if (nsplit > 1) part_acc[((t * nsplit + z) * H + h0 + hh) * r + d] = acc[c][hh];
+        else out[(t * H + h0 + hh) * r + d] = acc[c][hh] / l * f;
+      }
     }
   }
   if (nsplit > 1 && tid < nh) {
@@ -576,34 +620,46 @@ __global__ void __launch_bounds__(kAttnThreads) latent_window_attn_kernel(
   }
 }
 
-// out[t, h, :] = sum_z w_z acc_z / sum_z w_z l_z with w_z = exp(m_z - max_z m_z); pieces without keys have l_z = 0
-__global__ void __launch_bounds__(128) latent_attn_combine_kernel(const float* __restrict__ part_acc, const float* __restrict__ part_ml,
+// out[t, h, :] = sum_z w_z acc_z / sum_z w_z l_z with w_z = exp(m_z - max_z m_z); pieces without keys have l_z = 0, hold zeros and get the
+// weight 0, so that no load waits for a branch
+__global__ void __launch_bounds__(512) latent_attn_combine_kernel(const float* __restrict__ part_acc, const float* __restrict__ part_ml,
                                                                   int H, int r, int nsplit, float* __restrict__ out,
                                                                   const int* __restrict__ seq_of, const int* __restrict__ cu, int skip_from,
                                                                   const float* __restrict__ gate, long long ldg) {
+  extern __shared__ float wz[];           // [nsplit]
+  __shared__ float red[32];
   const long long t = blockIdx.x;
   const int h = blockIdx.y;
   if (cu != nullptr) {
     const int sq = seq_of[t];
     if (cu[sq + 1] - cu[sq] >= skip_from) return;
   }
+  auto ml = [&](int z) { return *reinterpret_cast<const float2*>(part_ml + ((t * nsplit + z) * H + h) * 2); };
   float M = -INFINITY;
-  for (int zz = 0; zz < nsplit; ++zz) {
-    const float* ml = part_ml + ((t * nsplit + zz) * H + h) * 2;
-    if (ml[1] > 0.f) M = fmaxf(M, ml[0]);
+  for (int z = threadIdx.x; z < nsplit; z += blockDim.x) {
+    const float2 v = ml(z);
+    if (v.y > 0.f) M = fmaxf(M, v.x);
   }
+  M = warp_max(M);
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = M;
+  __syncthreads();
+  for (int w = 0; w < (int)blockDim.x >> 5; ++w) M = fmaxf(M, red[w]);
   float L = 0.f;
-  for (int zz = 0; zz < nsplit; ++zz) {
-    const float* ml = part_ml + ((t * nsplit + zz) * H + h) * 2;
-    if (ml[1] > 0.f) L += ml[1] * expf(ml[0] - M);
+  for (int z = threadIdx.x; z < nsplit; z += blockDim.x) {
+    const float2 v = ml(z);
+    const float w = v.y > 0.f ? expf(v.x - M) : 0.f;
+    wz[z] = w;
+    L = fmaf(w, v.y, L);
   }
+  L = block_sum(L, red);
+  const float f = head_gate(gate, ldg, t, h) / L;
+  const float* pa = part_acc + (t * nsplit * H + h) * r;
+  const long long step = (long long)H * r;
   for (int d = threadIdx.x; d < r; d += blockDim.x) {
     float v = 0.f;
-    for (int zz = 0; zz < nsplit; ++zz) {
-      const float* ml = part_ml + ((t * nsplit + zz) * H + h) * 2;
-      if (ml[1] > 0.f) v = fmaf(part_acc[((t * nsplit + zz) * H + h) * r + d], expf(ml[0] - M), v);
-    }
-    out[(t * H + h) * r + d] = v / L * head_gate(gate, ldg, t, h);
+#pragma unroll 8
+    for (int z = 0; z < nsplit; ++z) v = fmaf(wz[z], pa[z * step + d], v);
+    out[(t * H + h) * r + d] = v * f;
   }
 }
 
@@ -1091,23 +1147,34 @@ KB2SEQ_API int kb2_seq_latent_window_attn(const float* q_abs, const float* proj,
       window <= 0 || bad_dt(dt_cache))
     return failf(KB2SEQ_ERR_VALUE, "latent_window_attn: bad argument");
   if (r > kAttnThreads * kAttnAcc) return failf(KB2SEQ_ERR_VALUE, "latent_window_attn: latent size %d > %d", r, kAttnThreads * kAttnAcc);
-  int HG = 8;                              // heads per block: a power of two, so that the 8 warps split evenly over the heads
-  while (HG > 1 && (HG > H || HG * r > kAttnThreads * kAttnAcc)) HG >>= 1;
   const int D = r + dr;
-  const int KT = 32;
-  auto smem_of = [&](int hg, int kt) { return (size_t)(hg * D + kt * (D + 1) + hg * kt + 8 * kt + 3 * hg) * 4 + (size_t)kt * 8; };
-  while (HG > 1 && smem_of(HG, KT) > 200 * 1024) HG >>= 1;
+  int NC = 1;                              // latent columns per thread: a power of two
+  while (NC * kAttnThreads < r) NC <<= 1;
+  int HG = 8;                              // heads per block: a power of two, HG x NC sums per thread
+  while (HG > 1 && (HG > H || HG * NC > kAttnAcc || attn_smem_floats(HG, D) * 4 > 200 * 1024)) HG >>= 1;
   if (nsplit < 1 || nsplit > 1024 || (nsplit > 1 && (!part_acc || !part_ml))) return failf(KB2SEQ_ERR_VALUE, "latent_window_attn: bad key split");
-  const size_t smem = smem_of(HG, KT);
+  const size_t smem = attn_smem_floats(HG, D) * 4;
   if (smem > 200 * 1024) return failf(KB2SEQ_ERR_VALUE, "latent_window_attn: latent + rotated size %d too large", D);
-  if (smem > 48 * 1024) SEQ_CUDA(cudaFuncSetAttribute(latent_window_attn_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-  dim3 grid(T, (H + HG - 1) / HG, nsplit);
-  latent_window_attn_kernel<<<grid, kAttnThreads, smem, (cudaStream_t)stream>>>(q_abs, proj, ldp, H, HG, dn, dr, r, ckv, kr, dt_cache, positions,
-                                                                                 seq_of, pages, max_pages, page_size, sinks, scale, window, KT,
-                                                                                 out, cu, skip_from, nsplit, part_acc, part_ml, gate, ldg);
+  const dim3 grid(T, (H + HG - 1) / HG, nsplit);
+#define KB2_LA(HGV, NCV)                                                                                                                      \
+  case HGV * 32 + NCV: {                                                                                                                      \
+    if (smem > 48 * 1024)                                                                                                                     \
+      SEQ_CUDA(cudaFuncSetAttribute(latent_window_attn_kernel<HGV, NCV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));            \
+    latent_window_attn_kernel<HGV, NCV><<<grid, kAttnThreads, smem, (cudaStream_t)stream>>>(                                                   \
+        q_abs, proj, ldp, H, dn, dr, r, ckv, kr, dt_cache, positions, seq_of, pages, max_pages, page_size, sinks, scale, window, out, cu,     \
+        skip_from, nsplit, part_acc, part_ml, gate, ldg);                                                                                     \
+    break;                                                                                                                                    \
+  }
+  switch (HG * 32 + NC) {
+    KB2_LA(8, 1) KB2_LA(8, 2) KB2_LA(4, 1) KB2_LA(4, 2) KB2_LA(4, 4) KB2_LA(2, 1) KB2_LA(2, 2) KB2_LA(2, 4) KB2_LA(2, 8)
+    KB2_LA(1, 1) KB2_LA(1, 2) KB2_LA(1, 4) KB2_LA(1, 8) KB2_LA(1, 16)
+    default: return failf(KB2SEQ_ERR_VALUE, "latent_window_attn: no kernel for %d heads x %d columns", HG, NC);
+  }
+#undef KB2_LA
   SEQ_LAUNCHED();
   if (nsplit > 1) {
-    latent_attn_combine_kernel<<<dim3(T, H), 128, 0, (cudaStream_t)stream>>>(part_acc, part_ml, H, r, nsplit, out, seq_of, cu, skip_from, gate, ldg);
+    latent_attn_combine_kernel<<<dim3(T, H), r >= 512 ? 512 : (r + 31) / 32 * 32, (size_t)nsplit * 4, (cudaStream_t)stream>>>(part_acc, part_ml, H, r, nsplit, out, seq_of, cu, skip_from,
+                                                                                               gate, ldg);
     SEQ_LAUNCHED();
   }
   return KB2SEQ_OK;
