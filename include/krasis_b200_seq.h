@@ -76,14 +76,20 @@ KB2SEQ_API int kb2_seq_latent_window_attn(const float* q_abs, const float* proj,
 KB2SEQ_API int kb2_seq_conv_silu(const float* proj, long long ldp, int T, int S, int C, int K, const float* taps, float* tail,
                                  const int* seq_of, const int* cu, const int* slots, float* out, void* stream);
 
-/* The same with a bias added to proj before the convolution (null: none; the carried tail holds biased inputs) and act 1: silu, 0: none.
- * act + 2: the bias joins the convolution's result instead of its inputs (ahead of the activation; the tail holds plain inputs). */
-KB2SEQ_API int kb2_seq_conv(const float* proj, long long ldp, int T, int S, int C, int K, const float* taps, const float* bias, int act,
-                            float* tail, const int* seq_of, const int* cu, const int* slots, float* out, void* stream);
+/* The same with a bias added to proj before the convolution (null: none; the carried tail holds biased inputs), a bias_out added to its
+ * result ahead of the activation (null: none), and act 1: silu, 0: none. */
+KB2SEQ_API int kb2_seq_conv(const float* proj, long long ldp, int T, int S, int C, int K, const float* taps, const float* bias,
+                            const float* bias_out, int act, float* tail, const int* seq_of, const int* cu, const int* slots, float* out,
+                            void* stream);
 
 /* x += y_mult * y (y may be null); h = x / sqrt(mean(x^2) + eps) * (w_shift + w) (h may be null; h == x with y null: in place, fp32) */
 KB2SEQ_API int kb2_seq_residual_scale_rms(float* x, const float* y, float y_mult, const float* w, float w_shift, void* h, int dt_h, int T,
                                           int W, float eps, void* stream);
+
+/* Norm on the sublayer's output only: z = c1 y1 + c2 y2 + bias (y2, bias [W] may be null), x += mult * z / sqrt(mean(z^2) + eps) * w, and,
+ * if h is given, h = x in dt_h or, with wh, x / sqrt(mean(x^2) + eps) * wh.  y1 null: x stays (h is then its rounded copy or its norm). */
+KB2SEQ_API int kb2_seq_residual_post_rms(float* x, const float* y1, float c1, const float* y2, float c2, const float* bias, float mult,
+                                         const float* w, const float* wh, void* h, int dt_h, int T, int W, float eps, void* stream);
 
 /* gated delta rule over each sequence's portion; state [slots][H][dk][dv] fp32 is read and written back.
  * scratch (fp32, 2 T Hk dk + 2 T H + T H dv + 4 elements, 16-byte aligned) selects the register-state kernels when dk is 32, 64 or
@@ -115,11 +121,13 @@ KB2SEQ_API int kb2_seq_residual_add_norm(float* x, const float* y, const float* 
  * back in place; k [G M d] and v [G dv] go to the cache rows of the tokens' positions.  norm_whole 1: one root mean square over the whole
  * of q (and of k) with weights qw [H M d] / kw [G M d].  rot_half 1: dimension i turns with i + rot_dims / 2 instead of 2i with 2i + 1.
  * vfreq [dv / 2] (may be null): the value vectors are cached rotated too, pair m of all dv dimensions (same pair layout) by
- * position * vfreq[m]; kb2_seq_attn_finish turns the attention output back by the query's position. */
+ * position * vfreq[m]; kb2_seq_attn_finish turns the attention output back by the query's position.  amp multiplies sin and cos of the
+ * query / key rotation.  v_is_k 1 (needs M == 1 and dv == d): there is no v in proj, the values are the keys with their bias, ahead of norm
+ * and rotation. */
 KB2SEQ_API int kb2_seq_head_kv_prep(float* proj, long long ldp, int T, int H, int G, int M, int d, int dv, const float* bias,
                                     const float* qw, const float* kw, float eps, const double* freq, int rot_dims, const int* positions,
                                     const int* seq_of, const int* pages, int max_pages, int page_size, void* kc, void* vc, int dt_cache,
-                                    int norm_whole, int rot_half, const double* vfreq, void* stream);
+                                    int norm_whole, int rot_half, const double* vfreq, float amp, int v_is_k, void* stream);
 
 /* Pooled blocks: every `pool` consecutive positions of a sequence, b pool .. b pool + pool - 1, are summarised by the mean of their
  * cached key rows (width kw) and the mean of their cached value rows (width vw), taken in fp32 from the cache as it holds them.  The
@@ -160,9 +168,12 @@ KB2SEQ_API int kb2_seq_attn_finish(const float* a, const float* part_acc, const 
                                    const int* positions, const double* vfreq, int rot_half, void* stream);
 
 /* in [rows, ld_in] = [gate: F | up: F]; out [rows, F].  kind 0: gelu_tanh(g) u, 1: silu(g) u, 2: g' sigmoid(alpha g') (u' + 1) with
- * g' = min(g, limit), u' = clamp(u, -limit, limit), 3: relu(g)^2 of in [rows, ld_in >= F] (no up half).  n_tiles (device, may be null): only n_tiles[0] * tile_rows rows are computed. */
+ * g' = min(g, limit), u' = clamp(u, -limit, limit), 3: relu(g)^2 of in [rows, ld_in >= F] (no up half).  n_tiles (device, may be null): only n_tiles[0] * tile_rows rows are computed.
+ * row_w (may be null): both halves are first multiplied by row_w[r], or with row_map by row_w[row_map[r]] (negative entry: 0).  bias
+ * (may be null) [2 F] (kind 3: [F]) is then added. */
 KB2SEQ_API int kb2_seq_glu(const void* in, int dt_in, long long ld_in, void* out, int dt_out, long long rows, int F, int kind, float limit,
-                           float alpha, const int* n_tiles, int tile_rows, void* stream);
+                           float alpha, const int* n_tiles, int tile_rows, const float* bias, const float* row_w, const int* row_map,
+                           void* stream);
 
 /* Router: z [T, ldz] fp32 logits of E outputs (bias [E], may be null, is added first) -> ids [T, top], weights [T, top].
  * score_kind 0 softmax, 1 sigmoid, 2 the logit itself (weights are then the softmax over the chosen logits alone); choice = score +
@@ -188,7 +199,7 @@ KB2SEQ_API int kb2_seq_moe_gemm(const void* A, int dtA, long long lda, const int
 KB2SEQ_API int kb2_seq_moe_gemv(const void* A, int dtA, long long lda, int div, const int* ids, int E, const void* B, int dtB, long long ldb,
                                 long long sB, void* C, int dtC, long long ldc, int slots, int N, int K, void* stream);
 /* out[t, :] = sum_k weights[t, k] * (y[row of slot (t, k)] | h[t] if E <= ids < E + ident) + f shared[t] (may be null); pos_of_slot null:
- * the row of a slot is the slot itself.  f = sigmoid(shared_gate[t * ldsg]), or 1 when shared_gate is null. */
+ * the row of a slot is the slot itself; weights null (needs ident 0): ones.  f = sigmoid(shared_gate[t * ldsg]), or 1 when shared_gate is null. */
 KB2SEQ_API int kb2_seq_moe_combine(const float* y, const int* pos_of_slot, const int* ids, const float* weights, int T, int top, int E,
                                    int ident, const void* h, int dt_h, const float* shared, float* out, int W, const float* shared_gate,
                                    long long ldsg, void* stream);
@@ -205,6 +216,31 @@ KB2SEQ_API int kb2_seq_gla(const float* qkv, long long ld, int q_off, int k_off,
                            const float* decay_bias, float tau, float q_scale, int T, int S, int H, int dk, int dv, float* state,
                            const int* cu, const int* slots, float* scratch, float* out, void* stream);
 
+/* Matrix memory (mLSTM) over each sequence's portion.  proj [T, ld] fp32 holds q and k (H x dk columns from q_off / k_off; q is multiplied by
+ * q_scale), v (H x dv from v_off) and the gate inputs (H columns from i_off / f_off, plus i_bias / f_bias [H], which may be null).  Per head
+ *   i = cap tanh(z_i / cap), f = logsigmoid(cap tanh(z_f / cap)), m_t = max(f + m_(t-1), i),
+ *   S <- exp(f + m_(t-1) - m_t) S + exp(i - m_t) k v^T, n likewise with k alone, m_0 = 0:
+ * out [T, H dv] = S^T q (fp32) and den [T, H] = max(|n . q|, exp(-m)) + 1e-6; kb2_seq_head_norm_gate divides and finishes.
+ * state [slots][H][dk][dv], nstate [slots][H][dk] and mstate [slots][H] (fp32) are read and written back.  scratch: 3 T H fp32 elements.
+ * Key sizes 32 / 64 / 128 / 256 with value sizes that are multiples of 32 (and 16-byte rows and offsets) keep the state in registers;
+ * others run a generic kernel (dk <= 1024, any dv). */
+KB2SEQ_API int kb2_seq_mlstm(const float* proj, long long ld, int q_off, int k_off, int v_off, int i_off, int f_off, const float* i_bias,
+                             const float* f_bias, float cap, float q_scale, int T, int S, int H, int dk, int dv, float* state, float* nstate,
+                             float* mstate, const int* cu, const int* slots, float* scratch, float* out, float* den, void* stream);
+
+/* Real-gated linear recurrent unit over each sequence's portion, C channels in blocks of bs.  u [T, ldu]: inputs; z: gate products, the
+ * pair of channel c = b bs + j of token t at z[t ldz + b zb + j] (recurrence gate r) and z[t ldz + b zb + bs + j] (input gate i);
+ * y [T, ldy]: the other branch; biases [C] may be null.  log a = -8 sigmoid(r) softplus(lam), S <- a S + sqrt(1 - a^2) sigmoid(i) u,
+ * out [T, C] = S gelu_tanh(y) in dt_out; state [slots][C] fp32 is read and written back. */
+KB2SEQ_API int kb2_seq_rglru(const float* u, long long ldu, const float* z, long long ldz, long long zb, const float* y, long long ldy,
+                             const float* r_bias, const float* i_bias, const float* y_bias, const float* lam, int T, int S, int C, int bs,
+                             float* state, const int* cu, const int* slots, void* out, int dt_out, void* stream);
+
+/* out [blocks][T_pad][2 bs] bf16: row (b, t) = [high | low] parts of u[t, b bs .. b bs + bs), whose sum is the fp32 value to 2^-17 of its
+ * size; rows t >= T are left as they are.  With weights [W_b | W_b] per block the grouped tensor-core product is a block-diagonal product
+ * of the fp32 rows.  bs even. */
+KB2SEQ_API int kb2_seq_split_blocks(const float* u, long long ldu, int T, int T_pad, int blocks, int bs, void* out, void* stream);
+
 /* Selective scan over each sequence's portion: per channel c and state n, S[c, n] <- exp(dt_c A[c, n]) S[c, n] + dt_c x_c B_n,
  * y_c = sum_n S[c, n] C_n + D[c] x_c, out = y_c silu(z_c), with dt = softplus(dt_in + dt_bias), A = -exp(A_log [inner, N]).
  * x [T, ldx], dt_in [T, ldd], bc [T, ldb] = [B: N | C: N] from column b_off, z [T, ldz] from column z_off, all fp32.
@@ -214,10 +250,11 @@ KB2SEQ_API int kb2_seq_selective_scan(const float* x, long long ldx, const float
                                       const float* D, int T, int S, int inner, int N, float* state, const int* cu, const int* slots,
                                       void* out, int dt_out, void* stream);
 
-/* out[t, h, :] = o[t, h, :] (o [T, ldo] fp32, H x dv columns), divided by its root mean square and times w [dv] if w is given, times
+/* out[t, h, :] = o[t, h, :] (o [T, ldo] fp32, H x dv columns), divided by den[t, h] if den [T, H] is given, divided by its root mean square
+ * and times w [dv] (w_heads 1: w [H dv], weights of their own for every head) if w is given, times
  * silu (gate_act 0) or sigmoid (1) of gate[t * ldg + h dv + :] if gate is given; out [T, H dv] in dt_out. */
 KB2SEQ_API int kb2_seq_head_norm_gate(const float* o, long long ldo, const float* w, float eps, const float* gate, long long ldg, int gate_act,
-                                      int T, int H, int dv, void* out, int dt_out, void* stream);
+                                      int T, int H, int dv, void* out, int dt_out, const float* den, int w_heads, void* stream);
 
 /* out[t, :n] = in[t, :n] / sqrt(mean(in[t, :n]^2) + eps) * w; in fp32 with row stride ld_in, out in dt_out with row stride ld_out */
 KB2SEQ_API int kb2_seq_rms_rows(const float* in, long long ld_in, int n, const float* w, float eps, void* out, int dt_out, long long ld_out,

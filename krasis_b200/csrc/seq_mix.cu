@@ -4,7 +4,8 @@
 //   head_kv_prep           bias, RMS norm (per vector, or one over the whole of q and one over the whole of k) and rotary positions
 //                          (pairs 2i / 2i + 1, or i / i + dims / 2) on the query and key vectors of every head and map; keys and
 //                          values go to the paged cache rows of the tokens' positions; optionally the values are rotated by their
-//                          positions over all of their dimensions
+//                          positions over all of their dimensions, or are the keys themselves as projected; optional amplitude of
+//                          the rotation
 //   kv_pool                the tokens that complete a block of `pool` positions write the mean of the block's cached keys and values
 //                          into pooled pools that share the page numbering
 //   paged_attn             softmax attention of every (head, map) query vector over the cached keys of its key/value head; the maps of
@@ -17,7 +18,8 @@
 //   attn_finish            merges the pieces, combines the maps with per-map coefficients (differential attention: 1, -lambda),
 //                          unit RMS norm per head, turning rotated values back by the query's position, output gate sigmoid(g) per
 //                          head or per element
-//   glu                    act(gate) * up in three flavours (tanh-GELU, SiLU, clamped swish with up + 1), or relu^2 without an up half
+//   glu                    act(gate) * up in three flavours (tanh-GELU, SiLU, clamped swish with up + 1), or relu^2 without an up half;
+//                          optional bias on both halves, optional weight per row on the unit's input
 //   route_topk             logits (+ bias) -> scores (softmax, sigmoid, or the logits themselves) -> + correction -> best groups (by their
 //                          best or two best members) -> top-k -> weights (the scores, or a softmax over the chosen logits alone)
 //   moe_bin / moe_gemm / moe_gemv / moe_combine
@@ -41,7 +43,8 @@ __global__ void __launch_bounds__(256) head_kv_prep_kernel(float* __restrict__ p
                                                            int rot_dims, const int* __restrict__ positions,
                                                            const int* __restrict__ seq_of, const int* __restrict__ pages, int max_pages,
                                                            int page_size, void* __restrict__ kc, void* __restrict__ vc, int dt_cache,
-                                                           int norm_whole, int rot_half, const double* __restrict__ vfreq) {
+                                                           int norm_whole, int rot_half, const double* __restrict__ vfreq, float amp,
+                                                           int v_is_k) {
   extern __shared__ float rot_tab[];          // [rot_dims / 2][2]: cos, sin of the token's position, shared by all its vectors
   __shared__ float red[32];
   const long long t = blockIdx.x;
@@ -50,7 +53,7 @@ __global__ void __launch_bounds__(256) head_kv_prep_kernel(float* __restrict__ p
   const long long slot = (long long)pages[(long long)seq_of[t] * max_pages + pos / page_size] * page_size + pos % page_size;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
   const int nq = H * M, nvec = (H + G) * M, half = rot_dims >> 1;
-  for (int j = threadIdx.x; j < half; j += blockDim.x) rot_cs(pos, freq[j], 1.f, &rot_tab[2 * j], &rot_tab[2 * j + 1]);
+  for (int j = threadIdx.x; j < half; j += blockDim.x) rot_cs(pos, freq[j], amp, &rot_tab[2 * j], &rot_tab[2 * j + 1]);
   float rstd_q = 1.f, rstd_k = 1.f;
   if (norm_whole) {
     const int nqe = nq * d, nke = (nvec - nq) * d;
@@ -109,7 +112,7 @@ __global__ void __launch_bounds__(256) head_kv_prep_kernel(float* __restrict__ p
       if (is_q) x[i] = v; else st_dt(kc, dt_cache, krow + i, v);
     }
   }
-  const long long v0 = (long long)nvec * d;
+  const long long v0 = (long long)(v_is_k ? nq : nvec) * d;      // values that are the keys as projected (biased), ahead of norm and rotation
   if (vfreq == nullptr) {
     for (int i = threadIdx.x; i < G * dv; i += blockDim.x)
       st_dt(vc, dt_cache, slot * G * dv + i, p[v0 + i] + (bias ? bias[v0 + i] : 0.f));
@@ -445,7 +448,8 @@ __global__ void __launch_bounds__(256) pool_merge_kernel(float* __restrict__ a, 
 }
 
 // ------------------------------------------------------------------------------------------------ gated linear units
-// in [rows, 2 F] = [gate | up].  kind 0: gelu_tanh(g) u; 1: silu(g) u; 2: g' sigmoid(alpha g') (u' + 1) with g' = min(g, limit),
+// in [rows, 2 F] = [gate | up], first times row_w[row] (a weight on the unit's input: the two products are linear in it; with row_map the
+// weight of row r is row_w[row_map[r]], 0 for a negative entry), then plus bias [2 F].  kind 0: gelu_tanh(g) u; 1: silu(g) u; 2: g' sigmoid(alpha g') (u' + 1) with g' = min(g, limit),
 // u' = clamp(u, -limit, limit); 3: relu(g)^2 of in [rows, F] alone (no up half).  With n_tiles given only the first
 // n_tiles[0] * tile_rows rows are computed.
 __device__ __forceinline__ float glu_value(float g, float u, int kind, float limit, float alpha) {
@@ -456,29 +460,57 @@ __device__ __forceinline__ float glu_value(float g, float u, int kind, float lim
   u = fminf(fmaxf(u, -limit), limit);
   return g / (1.f + expf(-alpha * g)) * (u + 1.f);
 }
+__device__ __forceinline__ float glu_row_weight(const float* __restrict__ row_w, const int* __restrict__ row_map, long long r) {
+  if (row_w == nullptr) return 1.f;
+  const long long i = row_map != nullptr ? row_map[r] : r;
+  return i < 0 ? 0.f : row_w[i];
+}
 __global__ void glu_kernel(const void* __restrict__ in, int dt_in, long long ld_in, void* __restrict__ out, int dt_out, long long rows, int F,
-                           int kind, float limit, float alpha, const int* __restrict__ n_tiles, int tile_rows) {
+                           int kind, float limit, float alpha, const int* __restrict__ n_tiles, int tile_rows, const float* __restrict__ bias,
+                           const float* __restrict__ row_w, const int* __restrict__ row_map) {
   if (n_tiles != nullptr) rows = min(rows, (long long)n_tiles[0] * tile_rows);
   const long long n = rows * F;
   for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x) {
     const long long r = i / F;
     const int f = (int)(i - r * F);
-    st_dt(out, dt_out, i, glu_value(ld_dt(in, dt_in, r * ld_in + f), kind == 3 ? 0.f : ld_dt(in, dt_in, r * ld_in + F + f), kind, limit, alpha));
+    const float rw = glu_row_weight(row_w, row_map, r);
+    float g = ld_dt(in, dt_in, r * ld_in + f) * rw, u = kind == 3 ? 0.f : ld_dt(in, dt_in, r * ld_in + F + f) * rw;
+    if (bias != nullptr) {
+      g += bias[f];
+      if (kind != 3) u += bias[F + f];
+    }
+    st_dt(out, dt_out, i, glu_value(g, u, kind, limit, alpha));
   }
 }
 
 // bf16 in and out, F and ld_in multiples of 8: 16-byte accesses
 __global__ void glu_bf16x8_kernel(const bf16* __restrict__ in, long long ld_in, bf16* __restrict__ out, long long rows, int F, int kind, float limit,
-                                  float alpha, const int* __restrict__ n_tiles, int tile_rows) {
+                                  float alpha, const int* __restrict__ n_tiles, int tile_rows, const float* __restrict__ bias,
+                                  const float* __restrict__ row_w, const int* __restrict__ row_map) {
   if (n_tiles != nullptr) rows = min(rows, (long long)n_tiles[0] * tile_rows);
   const int F8 = F >> 3;
   const long long n = rows * F8;
   for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x) {
     const long long r = i / F8;
     const int f = (int)(i - r * F8) << 3;
-    float a[8], b[8];
+    float a[8], b[8] = {};
     unpack8(*reinterpret_cast<const uint4*>(in + r * ld_in + f), a);
     if (kind != 3) unpack8(*reinterpret_cast<const uint4*>(in + r * ld_in + F + f), b);
+    if (row_w != nullptr) {
+      const float rw = glu_row_weight(row_w, row_map, r);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) {
+        a[e] *= rw;
+        b[e] *= rw;
+      }
+    }
+    if (bias != nullptr) {
+#pragma unroll
+      for (int e = 0; e < 8; ++e) {
+        a[e] += bias[f + e];
+        if (kind != 3) b[e] += bias[F + f + e];
+      }
+    }
     uint4 o;
     __nv_bfloat162* po = reinterpret_cast<__nv_bfloat162*>(&o);
 #pragma unroll
@@ -736,7 +768,7 @@ __global__ void __launch_bounds__(256) moe_gemv_kernel(const TA* __restrict__ A,
 }
 
 // out[t, :] = sum_k w[t, k] * (expert row of slot (t, k) | h[t, :] for an identity expert) + sigmoid(shared_gate[t]) shared[t, :] (gate
-// null: 1), k in selection order
+// null: 1), k in selection order; weights null: ones (weights that already went into the experts' inputs)
 __global__ void moe_combine_kernel(const float* __restrict__ y, const int* __restrict__ pos_of_slot, const int* __restrict__ ids,
                                    const float* __restrict__ weights, int top, int E, int ident, const void* __restrict__ h, int dt_h,
                                    const float* __restrict__ shared, float* __restrict__ out, int W,
@@ -749,7 +781,7 @@ __global__ void moe_combine_kernel(const float* __restrict__ y, const int* __res
       for (int k = 0; k < top; ++k) {
         const long long slot = t * top + k;
         const int e = ids[slot];
-        const float w = weights[slot];
+        const float w = weights ? weights[slot] : 1.f;
         if (e >= 0 && e < E) {
           const long long p = pos_of_slot ? pos_of_slot[slot] : slot;
           const float4 r = *reinterpret_cast<const float4*>(y + p * W + d);
@@ -773,7 +805,7 @@ __global__ void moe_combine_kernel(const float* __restrict__ y, const int* __res
     for (int k = 0; k < top; ++k) {
       const long long slot = t * top + k;
       const int e = ids[slot];
-      const float w = weights[slot];
+      const float w = weights ? weights[slot] : 1.f;
       if (e >= 0 && e < E) {
         const long long p = pos_of_slot ? pos_of_slot[slot] : slot;
         v = fmaf(w, y[p * W + d], v);
@@ -795,14 +827,15 @@ extern "C" {
 KB2SEQ_API int kb2_seq_head_kv_prep(float* proj, long long ldp, int T, int H, int G, int M, int d, int dv, const float* bias,
                                     const float* qw, const float* kw, float eps, const double* freq, int rot_dims, const int* positions,
                                     const int* seq_of, const int* pages, int max_pages, int page_size, void* kc, void* vc, int dt_cache,
-                                    int norm_whole, int rot_half, const double* vfreq, void* stream) {
+                                    int norm_whole, int rot_half, const double* vfreq, float amp, int v_is_k, void* stream) {
+  if (v_is_k && (M != 1 || dv != d)) return failf(KB2SEQ_ERR_VALUE, "head_kv_prep: values that are the keys need one map and dv == d");
   if (vfreq && (dv & 1)) return failf(KB2SEQ_ERR_VALUE, "head_kv_prep: rotated values need an even value size");
   if (!proj || !positions || !seq_of || !pages || T <= 0 || H <= 0 || G < 0 || M <= 0 || d <= 0 || dv < 0 || rot_dims < 0 ||
       rot_dims > d || (rot_dims & 1) || (rot_dims && !freq) || page_size <= 0 || max_pages <= 0 || bad_dt(dt_cache) ||
       (G > 0 && (!kc || !vc)))
     return failf(KB2SEQ_ERR_VALUE, "head_kv_prep: bad argument");
   head_kv_prep_kernel<<<T, 256, (size_t)rot_dims * 4, (cudaStream_t)stream>>>(proj, ldp, H, G, M, d, dv, bias, qw, kw, eps, freq, rot_dims, positions, seq_of,
-                                                           pages, max_pages, page_size, kc, vc, dt_cache, norm_whole, rot_half, vfreq);
+                                                           pages, max_pages, page_size, kc, vc, dt_cache, norm_whole, rot_half, vfreq, amp, v_is_k);
   SEQ_LAUNCHED();
   return KB2SEQ_OK;
 }
@@ -882,19 +915,22 @@ KB2SEQ_API int kb2_seq_attn_finish(const float* a, const float* part_acc, const 
 }
 
 KB2SEQ_API int kb2_seq_glu(const void* in, int dt_in, long long ld_in, void* out, int dt_out, long long rows, int F, int kind, float limit,
-                           float alpha, const int* n_tiles, int tile_rows, void* stream) {
+                           float alpha, const int* n_tiles, int tile_rows, const float* bias, const float* row_w, const int* row_map,
+                           void* stream) {
   if (!in || !out || rows <= 0 || F <= 0 || ld_in < (kind == 3 ? F : 2 * F) || kind < 0 || kind > 3 || bad_dt(dt_in) || bad_dt(dt_out))
     return failf(KB2SEQ_ERR_VALUE, "glu: bad argument");
   if (dt_in == 1 && dt_out == 1 && F % 8 == 0 && ld_in % 8 == 0 && !((uintptr_t)in & 15) && !((uintptr_t)out & 15)) {
     const long long n8 = rows * (F / 8);
     const unsigned blocks8 = (unsigned)((n8 + 255) / 256 > 148 * 16 ? 148 * 16 : (n8 + 255) / 256);
-    glu_bf16x8_kernel<<<blocks8, 256, 0, (cudaStream_t)stream>>>((const bf16*)in, ld_in, (bf16*)out, rows, F, kind, limit, alpha, n_tiles, tile_rows);
+    glu_bf16x8_kernel<<<blocks8, 256, 0, (cudaStream_t)stream>>>((const bf16*)in, ld_in, (bf16*)out, rows, F, kind, limit, alpha, n_tiles, tile_rows, bias, row_w,
+                                                              row_map);
     SEQ_LAUNCHED();
     return KB2SEQ_OK;
   }
   const long long n = rows * F;
   const unsigned blocks = (unsigned)((n + 255) / 256 > 148 * 16 ? 148 * 16 : (n + 255) / 256);
-  glu_kernel<<<blocks, 256, 0, (cudaStream_t)stream>>>(in, dt_in, ld_in, out, dt_out, rows, F, kind, limit, alpha, n_tiles, tile_rows);
+  glu_kernel<<<blocks, 256, 0, (cudaStream_t)stream>>>(in, dt_in, ld_in, out, dt_out, rows, F, kind, limit, alpha, n_tiles, tile_rows, bias, row_w,
+                                                              row_map);
   SEQ_LAUNCHED();
   return KB2SEQ_OK;
 }
@@ -987,7 +1023,7 @@ KB2SEQ_API int kb2_seq_moe_gemv(const void* A, int dtA, long long lda, int div, 
 KB2SEQ_API int kb2_seq_moe_combine(const float* y, const int* pos_of_slot, const int* ids, const float* weights, int T, int top, int E,
                                    int ident, const void* h, int dt_h, const float* shared, float* out, int W, const float* shared_gate,
                                    long long ldsg, void* stream) {
-  if (!ids || !weights || !out || T <= 0 || top <= 0 || E < 0 || ident < 0 || W <= 0 || (E > 0 && !y) || (ident > 0 && (!h || bad_dt(dt_h))))
+  if (!ids || (!weights && ident > 0) || !out || T <= 0 || top <= 0 || E < 0 || ident < 0 || W <= 0 || (E > 0 && !y) || (ident > 0 && (!h || bad_dt(dt_h))))
     return failf(KB2SEQ_ERR_VALUE, "moe_combine: bad argument");
   moe_combine_kernel<<<T, 256, 0, (cudaStream_t)stream>>>(y, pos_of_slot, ids, weights, top, E, ident, h, dt_h, shared, out, W, shared_gate, ldsg);
   SEQ_LAUNCHED();

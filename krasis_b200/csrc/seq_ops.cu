@@ -6,6 +6,7 @@
 //   gemm_nt / gemv_nt      C = A B^T for any M, N, K; fp32 or bf16 operands, fp32 accumulation in a fixed K order per output
 //   residual_norm          x += norm(y) (+ x0);  h = layer_norm(x)                    (residual update fused with the next norm)
 //   residual_scale_rms     x += m y;  h = x / rms(x) * (shift + w)                    (the same for RMS norms and a residual multiplier)
+//   residual_post_rms      z = c1 y1 + c2 y2 + b;  x += m z / rms(z) * w;  h = x or x / rms(x) * wh   (norm on the sublayer's output only)
 //   act_mul                gelu_tanh(a) * b                                           (gated feed-forward)
 //   side_gate              gelu_tanh(g) * per-layer slice of a token table            (per-layer token input)
 //   latent_prep            RMS-normed latent + rotated shared key -> paged cache, rotary on the query's rotated part (any frequency
@@ -13,7 +14,7 @@
 //   latent_window_attn     absorbed-form latent attention over the page list: sliding window, softmax with an optional per-head sink,
 //                          optional sigmoid gate per head on the result
 //   conv_silu (+ state)    short causal convolution per channel over time with a carried tail, optional bias ahead of the taps or on
-//                          their result, then SiLU or nothing; conv_run reads every input once on long steps
+//                          their result (or both), then SiLU or nothing; conv_run reads every input once on long steps
 //   delta_rule             gated delta rule S <- g S; u = beta (v - S^T k); S += k u^T; o = S^T q, state in fp32 slots,
 //                          unit-norm q / k, per-head RMS norm of o with a SiLU or sigmoid gate; g is one decay per head, or one
 //                          per head and key channel (it then multiplies the rows of S)
@@ -341,6 +342,99 @@ __global__ void __launch_bounds__(256) residual_scale_rms_kernel(float* x, const
   for (int d = threadIdx.x; d < W; d += blockDim.x) st_dt(h, dt_h, row * W + d, rowbuf[d] * rstd * (w_shift + w[d]));
 }
 
+// Norm on the sublayer's output only; the next sublayer reads the residual stream as it is.  One block per token row:
+// z = c1 y1 + c2 y2 + bias (y2, bias may be null), x (fp32) += mult * z / sqrt(mean(z^2) + eps) * w; then, if h is given, h = x in dt_h, or
+// with wh x / sqrt(mean(x^2) + eps) * wh (the norm ahead of the head).  y1 == nullptr: x is left as it is.  V columns per access.
+template <int V>
+__global__ void __launch_bounds__(256) residual_post_rms_kernel(float* __restrict__ x, const float* __restrict__ y1, float c1,
+                                                                const float* __restrict__ y2, float c2, const float* __restrict__ bias,
+                                                                float mult, const float* __restrict__ w, const float* __restrict__ wh,
+                                                                void* __restrict__ h, int dt_h, int W, float eps) {
+  extern __shared__ __align__(16) float rowbuf[];
+  __shared__ float red[32];
+  const long long base = (long long)blockIdx.x * W;
+  auto load = [](const float* p, float* v) {
+    if constexpr (V == 4) {
+      const float4 f = *reinterpret_cast<const float4*>(p);
+      v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w;
+    } else {
+      v[0] = p[0];
+    }
+  };
+  auto store = [](float* p, const float* v) {
+    if constexpr (V == 4) *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+    else p[0] = v[0];
+  };
+  auto store_h = [&](int d, const float* v) {
+    if (dt_h == 0) {
+      store((float*)h + base + d, v);
+    } else if constexpr (V == 4) {
+      const __nv_bfloat162 lo = __floats2bfloat162_rn(v[0], v[1]), hi = __floats2bfloat162_rn(v[2], v[3]);
+      uint2 o;
+      o.x = *reinterpret_cast<const uint32_t*>(&lo);
+      o.y = *reinterpret_cast<const uint32_t*>(&hi);
+      *reinterpret_cast<uint2*>((bf16*)h + base + d) = o;
+    } else {
+      ((bf16*)h)[base + d] = __float2bfloat16_rn(v[0]);
+    }
+  };
+  float ss = 0.f, rstd = 0.f;
+  if (y1 != nullptr) {
+    for (int d = threadIdx.x * V; d < W; d += blockDim.x * V) {
+      float z[V];
+      load(y1 + base + d, z);
+#pragma unroll
+      for (int i = 0; i < V; ++i) z[i] *= c1;
+      if (y2 != nullptr) {
+        float t[V];
+        load(y2 + base + d, t);
+#pragma unroll
+        for (int i = 0; i < V; ++i) z[i] = fmaf(c2, t[i], z[i]);
+      }
+      if (bias != nullptr) {
+        float t[V];
+        load(bias + d, t);
+#pragma unroll
+        for (int i = 0; i < V; ++i) z[i] += t[i];
+      }
+      store(rowbuf + d, z);
+#pragma unroll
+      for (int i = 0; i < V; ++i) ss = fmaf(z[i], z[i], ss);
+    }
+    rstd = mult / sqrtf(block_sum(ss, red) / (float)W + eps);
+    ss = 0.f;
+  }
+  for (int d = threadIdx.x * V; d < W; d += blockDim.x * V) {        // a thread reads back the columns it wrote
+    float xv[V];
+    load(x + base + d, xv);
+    if (y1 != nullptr) {
+      float z[V], wv[V];
+      load(rowbuf + d, z);
+      load(w + d, wv);
+#pragma unroll
+      for (int i = 0; i < V; ++i) xv[i] = fmaf(z[i] * rstd, wv[i], xv[i]);
+      store(x + base + d, xv);
+    }
+    if (wh != nullptr) {
+      store(rowbuf + d, xv);
+#pragma unroll
+      for (int i = 0; i < V; ++i) ss = fmaf(xv[i], xv[i], ss);
+    } else if (h != nullptr) {
+      store_h(d, xv);
+    }
+  }
+  if (wh == nullptr || h == nullptr) return;
+  rstd = 1.f / sqrtf(block_sum(ss, red) / (float)W + eps);
+  for (int d = threadIdx.x * V; d < W; d += blockDim.x * V) {
+    float xv[V], wv[V];
+    load(rowbuf + d, xv);
+    load(wh + d, wv);
+#pragma unroll
+    for (int i = 0; i < V; ++i) xv[i] = xv[i] * rstd * wv[i];
+    store_h(d, xv);
+  }
+}
+
 // ------------------------------------------------------------------------------------------------ elementwise
 __global__ void act_mul_kernel(const void* __restrict__ in, int dt_in, void* __restrict__ out, int dt_out, long long T, int F) {
   const long long t = blockIdx.y;
@@ -664,13 +758,13 @@ __global__ void __launch_bounds__(512) latent_attn_combine_kernel(const float* _
 }
 
 // ------------------------------------------------------------------------------------------------ short convolution + delta rule
-// y[t, c] = act(sum_j taps[c, j] * x[i - (K - 1) + j, c]) with i the token's index in its portion and x = proj + bias (bias may be null);
-// act 1: silu, 0: none.  Inputs before the portion come from the sequence's carried tail (the last K - 1 inputs of earlier portions,
+// y[t, c] = act(bias_out[c] + sum_j taps[c, j] * x[i - (K - 1) + j, c]) with i the token's index in its portion and x = proj + bias (either
+// bias may be null); act 1: silu, 0: none.  Inputs before the portion come from the sequence's carried tail (the last K - 1 inputs of earlier portions,
 // bias included; zeros at the start of a sequence).
 __global__ void conv_silu_kernel(const float* __restrict__ proj, long long ldp, int C, int K, const float* __restrict__ taps,
                                  const float* __restrict__ tail, const int* __restrict__ seq_of, const int* __restrict__ cu,
                                  const int* __restrict__ slots, long long T, float* __restrict__ out, const float* __restrict__ bias,
-                                 int act, int bias_after) {
+                                 int act, const float* __restrict__ bias_out) {
   const long long t = blockIdx.y;
   const int c = blockIdx.x * blockDim.x + threadIdx.x;
   if (c >= C) return;
@@ -678,9 +772,8 @@ __global__ void conv_silu_kernel(const float* __restrict__ proj, long long ldp, 
   const int s = seq_of[t];
   const int i = (int)(t - cu[s]);
   const float* tl = tail + ((long long)slots[s] * C + c) * (K - 1);
-  const float bv = bias != nullptr ? bias[c] : 0.f;
-  const float b = bias_after ? 0.f : bv;       // bias_after: the bias joins the convolution's result, not its inputs
-  float acc = bias_after ? bv : 0.f;
+  const float b = bias != nullptr ? bias[c] : 0.f;
+  float acc = bias_out != nullptr ? bias_out[c] : 0.f;
   for (int j = 0; j < K; ++j) {
     const int src = i - (K - 1) + j;
     const float xv = src >= 0 ? proj[(t - i + src) * ldp + c] + b : tl[(K - 1) + src];
@@ -696,15 +789,14 @@ __global__ void __launch_bounds__(256) conv_run_kernel(const float* __restrict__
                                                        const float* __restrict__ taps, const float* __restrict__ tail,
                                                        const int* __restrict__ seq_of, const int* __restrict__ cu,
                                                        const int* __restrict__ slots, long long T, float* __restrict__ out,
-                                                       const float* __restrict__ bias, int act, int bias_after) {
+                                                       const float* __restrict__ bias, int act, const float* __restrict__ bias_out) {
   const int c = blockIdx.x * blockDim.x + threadIdx.x;
   if (c >= C) return;
   const long long r0 = (long long)blockIdx.y * kConvRun, r1 = min(T, r0 + kConvRun);
   float w[kConvMaxTaps], x[kConvMaxTaps] = {};     // x[j]: the input K - 1 - j rows back, x[K - 1] the current one
 #pragma unroll
   for (int j = 0; j < kConvMaxTaps; ++j) w[j] = j < K ? taps[(long long)c * K + j] : 0.f;
-  const float bv = bias != nullptr ? bias[c] : 0.f;
-  const float b = bias_after ? 0.f : bv, b_out = bias_after ? bv : 0.f;
+  const float b = bias != nullptr ? bias[c] : 0.f, b_out = bias_out != nullptr ? bias_out[c] : 0.f;
   int s = -1;
   for (long long t = r0; t < r1; ++t) {
     const int st = seq_of[t];
@@ -1180,23 +1272,22 @@ KB2SEQ_API int kb2_seq_latent_window_attn(const float* q_abs, const float* proj,
   return KB2SEQ_OK;
 }
 
-KB2SEQ_API int kb2_seq_conv(const float* proj, long long ldp, int T, int S, int C, int K, const float* taps, const float* bias, int act,
-                            float* tail, const int* seq_of, const int* cu, const int* slots, float* out, void* stream) {
-  const int bias_after = act >> 1;
-  act &= 1;
-  if (!proj || !taps || !tail || !seq_of || !cu || !slots || !out || T <= 0 || S <= 0 || C <= 0 || K <= 0 || bias_after > 1)
+KB2SEQ_API int kb2_seq_conv(const float* proj, long long ldp, int T, int S, int C, int K, const float* taps, const float* bias,
+                            const float* bias_out, int act, float* tail, const int* seq_of, const int* cu, const int* slots, float* out,
+                            void* stream) {
+  if (!proj || !taps || !tail || !seq_of || !cu || !slots || !out || T <= 0 || S <= 0 || C <= 0 || K <= 0 || act < 0 || act > 1)
     return failf(KB2SEQ_ERR_VALUE, "conv: bad argument");
   if (T > 65535) return failf(KB2SEQ_ERR_VALUE, "conv: more than 65535 rows in one step");
   if (T >= 4 * kConvRun && K <= kConvMaxTaps)
     conv_run_kernel<<<dim3((C + 255) / 256, (T + kConvRun - 1) / kConvRun), 256, 0, (cudaStream_t)stream>>>(proj, ldp, C, K, taps, tail, seq_of,
-                                                                                                          cu, slots, T, out, bias, act, bias_after);
+                                                                                                          cu, slots, T, out, bias, act, bias_out);
   else
     conv_silu_kernel<<<dim3((C + 255) / 256, T), 256, 0, (cudaStream_t)stream>>>(proj, ldp, C, K, taps, tail, seq_of, cu, slots, T, out, bias,
-                                                                                 act, bias_after);
+                                                                                 act, bias_out);
   SEQ_LAUNCHED();
   if (K > 1) {
     const long long m = (long long)S * C;
-    conv_tail_kernel<<<(unsigned)((m + 255) / 256), 256, 0, (cudaStream_t)stream>>>(proj, ldp, C, K, tail, cu, slots, S, bias_after ? nullptr : bias);
+    conv_tail_kernel<<<(unsigned)((m + 255) / 256), 256, 0, (cudaStream_t)stream>>>(proj, ldp, C, K, tail, cu, slots, S, bias);
     SEQ_LAUNCHED();
   }
   return KB2SEQ_OK;
@@ -1204,7 +1295,7 @@ KB2SEQ_API int kb2_seq_conv(const float* proj, long long ldp, int T, int S, int 
 
 KB2SEQ_API int kb2_seq_conv_silu(const float* proj, long long ldp, int T, int S, int C, int K, const float* taps, float* tail,
                                  const int* seq_of, const int* cu, const int* slots, float* out, void* stream) {
-  return kb2_seq_conv(proj, ldp, T, S, C, K, taps, nullptr, 1, tail, seq_of, cu, slots, out, stream);
+  return kb2_seq_conv(proj, ldp, T, S, C, K, taps, nullptr, nullptr, 1, tail, seq_of, cu, slots, out, stream);
 }
 
 KB2SEQ_API int kb2_seq_residual_scale_rms(float* x, const float* y, float y_mult, const float* w, float w_shift, void* h, int dt_h, int T,
@@ -1215,6 +1306,24 @@ KB2SEQ_API int kb2_seq_residual_scale_rms(float* x, const float* y, float y_mult
   if (smem > 200 * 1024) return failf(KB2SEQ_ERR_VALUE, "residual_scale_rms: width %d too large", W);
   if (smem > 48 * 1024) SEQ_CUDA(cudaFuncSetAttribute(residual_scale_rms_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
   residual_scale_rms_kernel<<<T, 256, smem, (cudaStream_t)stream>>>(x, y, y_mult, w, w_shift, h, dt_h, W, eps);
+  SEQ_LAUNCHED();
+  return KB2SEQ_OK;
+}
+
+KB2SEQ_API int kb2_seq_residual_post_rms(float* x, const float* y1, float c1, const float* y2, float c2, const float* bias, float mult,
+                                         const float* w, const float* wh, void* h, int dt_h, int T, int W, float eps, void* stream) {
+  if (!x || T <= 0 || W <= 0 || bad_dt(dt_h) || (y1 && !w) || (!y1 && (y2 || !h)) || (wh && !h) || h == (void*)x)
+    return failf(KB2SEQ_ERR_VALUE, "residual_post_rms: bad argument");
+  const size_t smem = (size_t)W * 4;
+  if (smem > 200 * 1024) return failf(KB2SEQ_ERR_VALUE, "residual_post_rms: width %d too large", W);
+  const uintptr_t all = (uintptr_t)x | (uintptr_t)y1 | (uintptr_t)y2 | (uintptr_t)bias | (uintptr_t)w | (uintptr_t)wh | (uintptr_t)h;
+  if (W % 4 == 0 && !(all & 15)) {
+    if (smem > 40 * 1024) SEQ_CUDA(cudaFuncSetAttribute(residual_post_rms_kernel<4>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    residual_post_rms_kernel<4><<<T, 256, smem, (cudaStream_t)stream>>>(x, y1, c1, y2, c2, bias, mult, w, wh, h, dt_h, W, eps);
+  } else {
+    if (smem > 40 * 1024) SEQ_CUDA(cudaFuncSetAttribute(residual_post_rms_kernel<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    residual_post_rms_kernel<1><<<T, 256, smem, (cudaStream_t)stream>>>(x, y1, c1, y2, c2, bias, mult, w, wh, h, dt_h, W, eps);
+  }
   SEQ_LAUNCHED();
   return KB2SEQ_OK;
 }

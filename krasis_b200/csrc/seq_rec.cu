@@ -5,9 +5,17 @@
 //                          channel alpha = sigmoid(z)^(1 / tau); the state of a (sequence, head, slice of value columns) lives in
 //                          registers: a generic form (P lanes share a column and each keeps dk / P of its rows) and, for key sizes
 //                          32 / 64 / 128 / 256, a form with lane = column, warp = slice of rows and cp.async token tiles
+//                          the same two kernels serve the matrix memory of mLSTM, S <- keep_t S + add_t k_t v_t^T with one pair of numbers per
+//                          token and head and a further column of ones whose read-out is the normaliser
+//   mlstm_gates            log gates of mLSTM and their running maximum m_t = max(f_t + m_(t-1), i_t) by a (sum, maximum) scan; keep and add
+//                          relative to m_t
+//   rglru_scan             real-gated linear recurrent unit: per channel S <- a_t S + sqrt(1 - a_t^2) i_t u_t, times gelu of the other branch;
+//                          warps own pieces of the time axis and meet once per tile
+//   split_blocks           fp32 rows as a bf16 high and low part side by side, grouped per block of channels: a block-diagonal product of
+//                          fp32 inputs on the tensor cores
 //   selective_scan         S[c, n] <- exp(dt_c A[c, n]) S[c, n] + dt_c x_c B_n, y_c = sum_n S[c, n] C_n + D_c x_c, times silu(z);
 //                          the lanes of a channel keep its states in registers; their pieces of y meet in shared memory once per tile
-//   head_norm_gate         per head: o / rms(o) * w (optional) times silu or sigmoid of a gate column (optional)
+//   head_norm_gate         per head: o (/ a divisor per head) / rms(o) * w (optional) times silu or sigmoid of a gate column (optional)
 //   rms_rows               RMS norm of a column range of strided fp32 rows
 //   branch_merge           c (a / rms(a) * wa + b / rms(b) * wb): two mixers that read the same input, each normed, averaged
 //   depth_mix              the residual stream as a learned weighted sum of the embedding output and every layer's result, fused with
@@ -28,12 +36,22 @@ __device__ __forceinline__ float softplus_f(float z) { return z > 20.f ? z : log
 // q, k [T, ld] (H x dk columns from q_off / k_off), v (H x dv from v_off), decay_in [T, lda] (H x dk logits, + decay_bias).
 // Block (sequence s, head h, slice of CB value columns).  Lane l of a warp: column l % CW, key slice p = l / CW of P = 32 / CW;
 // thread rows are i = p + P ii, ii < KR.  Tokens are staged kRecTok at a time as (alpha, k, q) triples in shared memory.
-template <int KR>
+// SC (matrix memory): alpha = keep[t, h] for all rows, the keys are multiplied by add[t, h], and column dv of ones keeps the key sum in
+// nstate [slots][H][dk]; its read-out becomes den[t, h] = max(|n . q|, exp(-mx[t, h])) + 1e-6.
+struct MemoryGates {
+  const float* keep;       // [T, H]
+  const float* add;
+  const float* mx;
+  float* nstate;
+  float* den;              // [T, H]
+};
+__device__ __forceinline__ float memory_den(float nq, float m) { return fmaxf(fabsf(nq), expf(-m)) + 1e-6f; }
+template <int KR, bool SC>
 __global__ void __launch_bounds__(kRecThreads) gla_scan_kernel(const float* __restrict__ qkv, long long ld, int q_off, int k_off, int v_off,
                                                                const float* __restrict__ decay_in, long long lda,
                                                                const float* __restrict__ decay_bias, float inv_tau, float q_scale, int H,
                                                                int dk, int dv, int P, float* __restrict__ state, const int* __restrict__ cu,
-                                                               const int* __restrict__ slots, float* __restrict__ out) {
+                                                               const int* __restrict__ slots, float* __restrict__ out, MemoryGates mg) {
   extern __shared__ __align__(16) float sm[];
   float4* akq = reinterpret_cast<float4*>(sm);              // [kRecTok][dk]
   const int CW = 32 / P, CB = (kRecThreads / 32) * CW;
@@ -41,14 +59,15 @@ __global__ void __launch_bounds__(kRecThreads) gla_scan_kernel(const float* __re
   const int s = blockIdx.x, h = blockIdx.y, c0 = blockIdx.z * CB;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int p = lane / CW, cl = warp * CW + lane % CW, c = c0 + cl;
-  const bool live = c < dv;
+  const bool ones = SC && c == dv, live = c < dv || ones;
   const int row0 = cu[s], n = cu[s + 1] - row0;
-  float* S = state + ((long long)slots[s] * H + h) * dk * dv;
+  float* S = ones ? mg.nstate + ((long long)slots[s] * H + h) * dk : state + ((long long)slots[s] * H + h) * dk * dv + c;
+  const int pitch = ones ? 1 : dv;
   float st[KR];
 #pragma unroll
   for (int ii = 0; ii < KR; ++ii) {
     const int i = p + P * ii;
-    st[ii] = (live && i < dk) ? S[(long long)i * dv + c] : 0.f;
+    st[ii] = (live && i < dk) ? S[(long long)i * pitch] : 0.f;
   }
   for (int t0 = 0; t0 < n; t0 += kRecTok) {
     const int nt = min(kRecTok, n - t0);
@@ -56,17 +75,22 @@ __global__ void __launch_bounds__(kRecThreads) gla_scan_kernel(const float* __re
     for (int e = tid; e < nt * dk; e += kRecThreads) {
       const int tt = e / dk, i = e - tt * dk;
       const long long t = row0 + t0 + tt;
-      const float z = decay_in[t * lda + h * dk + i] + (decay_bias ? decay_bias[h * dk + i] : 0.f);
       float4 f;
-      f.x = expf(-softplus_f(-z) * inv_tau);                // sigmoid(z)^(1 / tau)
       f.y = qkv[t * ld + k_off + h * dk + i];
+      if constexpr (SC) {
+        f.x = mg.keep[t * H + h];
+        f.y *= mg.add[t * H + h];
+      } else {
+        const float z = decay_in[t * lda + h * dk + i] + (decay_bias ? decay_bias[h * dk + i] : 0.f);
+        f.x = expf(-softplus_f(-z) * inv_tau);              // sigmoid(z)^(1 / tau)
+      }
       f.z = qkv[t * ld + q_off + h * dk + i] * q_scale;
       f.w = 0.f;
       akq[e] = f;
     }
     for (int e = tid; e < nt * CB; e += kRecThreads) {
       const int tt = e / CB, cc = e - tt * CB;
-      vs[e] = c0 + cc < dv ? qkv[(long long)(row0 + t0 + tt) * ld + v_off + h * dv + c0 + cc] : 0.f;
+      vs[e] = c0 + cc < dv ? qkv[(long long)(row0 + t0 + tt) * ld + v_off + h * dv + c0 + cc] : (SC && c0 + cc == dv ? 1.f : 0.f);
     }
     __syncthreads();
     for (int tt = 0; tt < nt; ++tt) {
@@ -83,13 +107,17 @@ __global__ void __launch_bounds__(kRecThreads) gla_scan_kernel(const float* __re
         }
       }
       for (int off = CW; off < 32; off <<= 1) o += __shfl_xor_sync(0xffffffffu, o, off);
-      if (p == 0 && live) out[(long long)(row0 + t0 + tt) * H * dv + h * dv + c] = o;
+      const long long th = (long long)(row0 + t0 + tt) * H + h;
+      if (p == 0 && live) {
+        if (ones) mg.den[th] = memory_den(o, mg.mx[th]);
+        else out[th * dv + c] = o;
+      }
     }
   }
 #pragma unroll
   for (int ii = 0; ii < KR; ++ii) {
     const int i = p + P * ii;
-    if (live && i < dk) S[(long long)i * dv + c] = st[ii];
+    if (live && i < dk) S[(long long)i * pitch] = st[ii];
   }
 }
 
@@ -110,6 +138,9 @@ __global__ void gla_decay_kernel(const float* __restrict__ decay_in, long long l
 
 __device__ __forceinline__ void rec_cp_async16(void* smem_dst, const void* gmem_src) {
   asm volatile("cp.async.ca.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(smem_dst)), "l"(gmem_src) : "memory");
+}
+__device__ __forceinline__ void rec_cp_async4(void* smem_dst, const void* gmem_src) {
+  asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"((uint32_t)__cvta_generic_to_shared(smem_dst)), "l"(gmem_src) : "memory");
 }
 __device__ __forceinline__ void rec_cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
 __device__ __forceinline__ void rec_cp_async_wait_all() { asm volatile("cp.async.wait_group 0;" ::: "memory"); }
@@ -193,6 +224,273 @@ __global__ void __launch_bounds__(32 * kGlaWarps) gla_reg_kernel(const float* __
   for (int ii = 0; ii < Q; ++ii) Sg[(long long)(piece * Q + ii) * dv + j0 + lane] = S[ii];
 }
 
+// ------------------------------------------------------------------------------------------------ matrix memory (mLSTM)
+// Log gates per (token, head): i = cap tanh((zi + bi) / cap), f = logsigmoid(cap tanh((zf + bf) / cap)); the running maximum
+// m_t = max(f_t + m_(t-1), i_t); keep = exp(f_t + m_(t-1) - m_t), add = exp(i_t - m_t).  A block per (sequence, head), a thread per token
+// of the tile: (F, M) pairs compose as (F1 + F2, max(M1 + F2, M2)), so m_t = max(F + m_0, M) over the prefix.  Everything in fp64; m_t is
+// rounded to fp32 at every token and keep / add are taken relative to the rounded values: the matrix and its maximum agree exactly
+// wherever a prompt is cut, and the rounding of m cancels.
+constexpr int kGateThreads = 1024;
+__device__ __forceinline__ double softplus_d(double z) { return z > 40.0 ? z : log1p(exp(z)); }
+__global__ void __launch_bounds__(kGateThreads) mlstm_gates_kernel(const float* __restrict__ proj, long long ld, int i_off, int f_off,
+                                                                   const float* __restrict__ i_bias, const float* __restrict__ f_bias, float cap,
+                                                                   int H, float* __restrict__ mstate, const int* __restrict__ cu,
+                                                                   const int* __restrict__ slots, float* __restrict__ keep,
+                                                                   float* __restrict__ add, float* __restrict__ mx) {
+  __shared__ double wF[32], wM[32];
+  __shared__ float ms[kGateThreads + 1];             // ms[1 + k]: m of the tile's token k, ms[0]: m before the tile
+  const int s = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int t0 = cu[s], n = cu[s + 1] - t0;
+  float* mp = mstate + (long long)slots[s] * H + h;
+  const double c = cap, bi = i_bias ? i_bias[h] : 0.f, bf = f_bias ? f_bias[h] : 0.f;
+  float m0 = *mp;
+  for (int b0 = 0; b0 < n; b0 += blockDim.x) {
+    const int nt = min((int)blockDim.x, n - b0);
+    const long long t = t0 + b0 + tid;
+    double f = 0.0, i = -1e300;                      // a place without a token: the neutral pair
+    if (tid < nt) {
+      i = c * tanh(((double)proj[t * ld + i_off + h] + bi) / c);
+      f = -softplus_d(-c * tanh(((double)proj[t * ld + f_off + h] + bf) / c));
+    }
+    double F = f, M = i;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const double Fp = __shfl_up_sync(0xffffffffu, F, o), Mp = __shfl_up_sync(0xffffffffu, M, o);
+      if (lane >= o) {
+        M = fmax(Mp + F, M);
+        F += Fp;
+      }
+    }
+    if (lane == 31) {
+      wF[warp] = F;
+      wM[warp] = M;
+    }
+    if (tid == 0) ms[0] = m0;
+    __syncthreads();
+    double m = m0;                                   // the maximum ahead of this warp's first token
+    for (int w = 0; w < warp; ++w) m = fmax(wF[w] + m, wM[w]);
+    m = fmax(F + m, M);
+    ms[1 + tid] = (float)m;
+    __syncthreads();
+    if (tid < nt) {
+      const double prev = ms[tid], cur = ms[1 + tid];
+      keep[t * H + h] = (float)exp(f + prev - cur);
+      add[t * H + h] = (float)exp(i - cur);
+      mx[t * H + h] = ms[1 + tid];
+    }
+    m0 = ms[nt];
+    __syncthreads();
+  }
+  if (tid == 0) *mp = m0;
+}
+
+// two fp32 lanes of one 64-bit register (packed FMA of sm_100)
+__device__ __forceinline__ uint64_t pack2(float lo, float hi) {
+  uint64_t r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(lo), "f"(hi));
+  return r;
+}
+__device__ __forceinline__ float sum2(uint64_t v) {
+  float lo, hi;
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(v));
+  return lo + hi;
+}
+__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
+  uint64_t r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+  return r;
+}
+__device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
+  uint64_t r;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
+
+// The recurrence of the matrix memory with the layout of gla_reg: a block owns 32 value columns of a (sequence, head), lane = column, warp =
+// DK / 8 rows in registers, two rows per 64-bit register.  One decay per token and head, so k and q are all a token broadcasts; add joins
+// the value.  The last block of a head (blockIdx.z == dv / 32) keeps the key sum: its value is 1 and lane 0 stands for the column.
+template <int DK>
+__global__ void __launch_bounds__(32 * kGlaWarps) mlstm_reg_kernel(const float* __restrict__ qkv, long long ld, int q_off, int k_off, int v_off,
+                                                                   float q_scale, int H, int dv, float* __restrict__ state,
+                                                                   const int* __restrict__ cu, const int* __restrict__ slots,
+                                                                   float* __restrict__ out, MemoryGates mg) {
+  constexpr int P = kGlaWarps, NT = 32 * P, Q = DK / P;
+  extern __shared__ __align__(16) float sm[];
+  float* ks = sm;                                   // [2][kGlaTile][DK]
+  float* qs = ks + 2 * kGlaTile * DK;
+  float* vs = qs + 2 * kGlaTile * DK;               // [2][kGlaTile][32]
+  float* gs = vs + 2 * kGlaTile * 32;               // [2][kGlaTile][2]: keep, add
+  float* os_part = gs + 2 * kGlaTile * 2;           // [kGlaTile][P][32]
+  const int s = blockIdx.x, h = blockIdx.y, j0 = blockIdx.z * 32;
+  const bool ones = j0 >= dv;
+  const int tid = threadIdx.x, lane = tid & 31, piece = tid >> 5;
+  const int t0 = cu[s], n = cu[s + 1] - cu[s];
+  const long long head = (long long)slots[s] * H + h;
+  float* Sg = ones ? mg.nstate + head * DK : state + head * DK * dv + j0 + lane;
+  const int pitch = ones ? 1 : dv;
+  uint64_t S[Q / 2];
+#pragma unroll
+  for (int ii = 0; ii < Q / 2; ++ii)
+    S[ii] = pack2(Sg[(long long)(piece * Q + 2 * ii) * pitch], Sg[(long long)(piece * Q + 2 * ii + 1) * pitch]);
+
+  auto load_tile = [&](int buf, int b0) {
+    const int nt = min(kGlaTile, n - b0);
+    for (int c = tid; c < nt * (DK / 4); c += NT) {                  // 16-byte chunks of the k and q rows
+      const int tt = c / (DK / 4), cc = c - tt * (DK / 4);
+      const long long row = t0 + b0 + tt;
+      const int dst = (buf * kGlaTile + tt) * DK + cc * 4;
+      rec_cp_async16(ks + dst, qkv + row * ld + k_off + h * DK + cc * 4);
+      rec_cp_async16(qs + dst, qkv + row * ld + q_off + h * DK + cc * 4);
+    }
+    if (!ones)
+      for (int c = tid; c < nt * 8; c += NT) {
+        const int tt = c >> 3, cc = c & 7;
+        rec_cp_async16(vs + (buf * kGlaTile + tt) * 32 + cc * 4, qkv + (long long)(t0 + b0 + tt) * ld + v_off + h * dv + j0 + cc * 4);
+      }
+    if (tid < 2 * nt) rec_cp_async4(gs + buf * kGlaTile * 2 + tid, ((tid & 1) ? mg.add : mg.keep) + (long long)(t0 + b0 + (tid >> 1)) * H + h);
+    rec_cp_async_commit();
+  };
+
+  load_tile(0, 0);
+  int buf = 0;
+  for (int b0 = 0; b0 < n; b0 += kGlaTile, buf ^= 1) {
+    const int nt = min(kGlaTile, n - b0);
+    rec_cp_async_wait_all();
+    __syncthreads();                                  // tile `buf` is in place; everyone is done with the other buffer and with os_part
+    if (b0 + kGlaTile < n) load_tile(buf ^ 1, b0 + kGlaTile);
+    for (int tt = 0; tt < nt; ++tt) {
+      const int base = (buf * kGlaTile + tt) * DK + piece * Q;
+      const ulonglong2* k4 = reinterpret_cast<const ulonglong2*>(ks + base);
+      const ulonglong2* q4 = reinterpret_cast<const ulonglong2*>(qs + base);
+      const float2 g = *reinterpret_cast<const float2*>(gs + (buf * kGlaTile + tt) * 2);
+      const float vv = (ones ? 1.f : vs[(buf * kGlaTile + tt) * 32 + lane]) * g.y;
+      const uint64_t keep = pack2(g.x, g.x), v2 = pack2(vv, vv);
+      uint64_t a0 = 0, a1 = 0;
+#pragma unroll
+      for (int ii = 0; ii < Q / 4; ++ii) {
+        const ulonglong2 kr = k4[ii], qr = q4[ii];
+        S[2 * ii] = fma2(S[2 * ii], keep, mul2(kr.x, v2));
+        S[2 * ii + 1] = fma2(S[2 * ii + 1], keep, mul2(kr.y, v2));
+        a0 = fma2(S[2 * ii], qr.x, a0);
+        a1 = fma2(S[2 * ii + 1], qr.y, a1);
+      }
+      os_part[(tt * P + piece) * 32 + lane] = sum2(a0) + sum2(a1);
+    }
+    __syncthreads();
+    for (int i = tid; i < nt * 32; i += NT) {
+      const int tt = i >> 5, c = i & 31;
+      float o = 0.f;
+#pragma unroll
+      for (int p = 0; p < P; ++p) o += os_part[(tt * P + p) * 32 + c];
+      const long long th = (long long)(t0 + b0 + tt) * H + h;
+      if (!ones) out[th * dv + j0 + c] = o * q_scale;
+      else if (c == 0) mg.den[th] = memory_den(o * q_scale, mg.mx[th]);
+    }
+  }
+  if (ones && lane != 0) return;                       // every lane holds the key sum
+#pragma unroll
+  for (int ii = 0; ii < Q / 2; ++ii) {
+    float lo, hi;
+    asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(S[ii]));
+    Sg[(long long)(piece * Q + 2 * ii) * pitch] = lo;
+    Sg[(long long)(piece * Q + 2 * ii + 1) * pitch] = hi;
+  }
+}
+
+// ------------------------------------------------------------------------------------------------ real-gated linear recurrent unit
+// u [T, ldu]: convolved inputs of C channels in blocks of bs; z: gate products, the pair of channel c = b bs + j at z + t ldz + b zb + j
+// (recurrence gate) and + bs (input gate); y [T, ldy] the other branch.  Per channel
+//   log a = -8 sigmoid(z_r + r_bias) softplus(lam),  S <- a S + sqrt(1 - a^2) sigmoid(z_i + i_bias) u,  out = S gelu_tanh(y + y_bias).
+// a = 1 + expm1(log a) and 1 - a^2 = -expm1 (2 + expm1): exact where a is next to one.  A block owns 32 channels (lane = channel) of a
+// sequence; warp w takes tokens [4 w, 4 w + 4) of a tile of 4 kRgWarps, composes its (a, b) pairs from S = 0, and the warps' compositions meet
+// in shared memory once per tile.  The next tile's inputs are in registers before this one's are used.
+constexpr int kRgWarps = 16, kRgTok = 4;
+__device__ __forceinline__ float sigmoid_f(float z) { return 1.f / (1.f + expf(-z)); }
+__global__ void __launch_bounds__(32 * kRgWarps) rglru_scan_kernel(const float* __restrict__ u, long long ldu, const float* __restrict__ z,
+                                                                   long long ldz, long long zb, const float* __restrict__ y, long long ldy,
+                                                                   const float* __restrict__ r_bias, const float* __restrict__ i_bias,
+                                                                   const float* __restrict__ y_bias, const float* __restrict__ lam, int C, int bs,
+                                                                   float* __restrict__ state, const int* __restrict__ cu,
+                                                                   const int* __restrict__ slots, void* __restrict__ out, int dt_out) {
+  __shared__ float Aw[2][kRgWarps][32], Bw[2][kRgWarps][32];
+  const int s = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int c = blockIdx.y * 32 + lane;
+  const bool live = c < C;
+  const int row0 = cu[s], n = cu[s + 1] - row0;
+  float* Sp = state + (long long)slots[s] * C + c;
+  float carry = live ? *Sp : 0.f;
+  const float rb = live && r_bias ? r_bias[c] : 0.f, ib = live && i_bias ? i_bias[c] : 0.f, yb = live && y_bias ? y_bias[c] : 0.f;
+  const float rate = live ? (float)(-8.0 * softplus_d((double)lam[c])) : 0.f;
+  const int blk = live ? c / bs : 0;
+  const float* zc = z + blk * zb + (c - blk * bs);
+  struct In { float u, r, i, y; };
+  In cur[kRgTok], nxt[kRgTok];
+  auto load = [&](In* in, int b0) {
+#pragma unroll
+    for (int k = 0; k < kRgTok; ++k) {
+      const int tt = b0 + warp * kRgTok + k;
+      in[k] = {0.f, 0.f, 0.f, 0.f};
+      if (live && tt < n) {
+        const long long t = row0 + tt;
+        in[k] = {u[t * ldu + c], zc[t * ldz], zc[t * ldz + bs], y[t * ldy + c]};
+      }
+    }
+  };
+  load(cur, 0);
+  int buf = 0;
+  for (int b0 = 0; b0 < n; b0 += kRgWarps * kRgTok, buf ^= 1) {
+    if (b0 + kRgWarps * kRgTok < n) load(nxt, b0 + kRgWarps * kRgTok);
+    float a[kRgTok], b[kRgTok], A = 1.f, B = 0.f;
+#pragma unroll
+    for (int k = 0; k < kRgTok; ++k) {
+      a[k] = 1.f;                                     // a place without a token leaves the state as it is
+      b[k] = 0.f;
+      if (live && b0 + warp * kRgTok + k < n) {
+        const float e = expm1f(rate * sigmoid_f(cur[k].r + rb));
+        a[k] = 1.f + e;
+        b[k] = sqrtf(-e * (2.f + e)) * sigmoid_f(cur[k].i + ib) * cur[k].u;
+      }
+      A *= a[k];
+      B = fmaf(a[k], B, b[k]);
+    }
+    Aw[buf][warp][lane] = A;
+    Bw[buf][warp][lane] = B;
+    __syncthreads();                                  // one barrier per tile: the other buffer is written only after the next one
+    float S = carry, mine = carry;
+#pragma unroll
+    for (int w = 0; w < kRgWarps; ++w) {
+      if (w == warp) mine = S;
+      S = fmaf(Aw[buf][w][lane], S, Bw[buf][w][lane]);
+    }
+    carry = S;
+#pragma unroll
+    for (int k = 0; k < kRgTok; ++k) {
+      const int tt = b0 + warp * kRgTok + k;
+      mine = fmaf(a[k], mine, b[k]);
+      if (live && tt < n) st_dt(out, dt_out, (long long)(row0 + tt) * C + c, mine * gelu_tanh(cur[k].y + yb));
+      cur[k] = nxt[k];
+    }
+  }
+  if (warp == 0 && live) *Sp = carry;
+}
+
+// u [T, ldu] fp32 -> out [blocks][Tp][2 bs] bf16: row (b, t) holds the channels of block b as [high | low], high + low = u up to 2^-17 |u|
+__global__ void __launch_bounds__(256) split_blocks_kernel(const float* __restrict__ u, long long ldu, long long T, long long Tp, int blocks, int bs,
+                                                           bf16* __restrict__ out) {
+  const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;     // a pair of channels
+  const int half = bs >> 1;
+  if (i >= T * blocks * half) return;
+  const long long t = i / (blocks * half);
+  const int r = (int)(i - t * blocks * half), b = r / half, j = (r - b * half) * 2;
+  const float v0 = u[t * ldu + b * bs + j], v1 = u[t * ldu + b * bs + j + 1];
+  const __nv_bfloat162 hi = __floats2bfloat162_rn(v0, v1);
+  const float2 back = __bfloat1622float2(hi);
+  const __nv_bfloat162 lo = __floats2bfloat162_rn(v0 - back.x, v1 - back.y);
+  bf16* row = out + (b * Tp + t) * 2 * bs + j;
+  *reinterpret_cast<__nv_bfloat162*>(row) = hi;
+  *reinterpret_cast<__nv_bfloat162*>(row + bs) = lo;
+}
+
 // ------------------------------------------------------------------------------------------------ selective scan
 // x [T, ldx] (inner channels after convolution and activation), dt_in [T, ldd] (+ dt_bias, then softplus), bc [T, ldb] = [B: N | C: N]
 // from b_off, z [T, ldz] from z_off, A_log [inner, N], D [inner].  Block (sequence, group of CB channels); lane l: state slice
@@ -201,9 +499,6 @@ __device__ __forceinline__ float ex2_approx_ftz(float x) {       // 2^x, MUFU.EX
   float y;
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
-}
-__device__ __forceinline__ void rec_cp_async4(void* smem_dst, const void* gmem_src) {
-  asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"((uint32_t)__cvta_generic_to_shared(smem_dst)), "l"(gmem_src) : "memory");
 }
 
 // Tiles of kRecTok tokens arrive by cp.async, double-buffered (dt input, x, z of the block's channels; B and C of the token), so that
@@ -314,22 +609,29 @@ __global__ void __launch_bounds__(kRecThreads) selective_scan_kernel(const float
 }
 
 // ------------------------------------------------------------------------------------------------ row kernels
-// out[t, h, :] = o[t, h, :] (/ rms * w[:] if w) (* act(gate[t, h dv + :]) if gate); a warp per (token, head).  gate_act 0: silu, 1: sigmoid
+// out[t, h, :] = o[t, h, :] (/ den[t, h]) (/ rms * w[:] if w) (* act(gate[t, h dv + :]) if gate); a warp per (token, head).  gate_act 0: silu,
+// 1: sigmoid.  w_heads: w [H dv], weights of their own for every head
 __global__ void __launch_bounds__(256) head_norm_gate_kernel(const float* __restrict__ o, long long ldo, const float* __restrict__ w, float eps,
                                                              const float* __restrict__ gate, long long ldg, int gate_act, int H, int dv,
-                                                             long long T, void* __restrict__ out, int dt_out) {
+                                                             long long T, void* __restrict__ out, int dt_out,
+                                                             const float* __restrict__ den, int w_heads) {
   const long long wi = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
   const int lane = threadIdx.x & 31;
   if (wi >= T * H) return;
   const long long t = wi / H;
   const int h = (int)(wi - t * H);
   const float* row = o + t * ldo + (long long)h * dv;
-  float rstd = 1.f;
+  const float dinv = den != nullptr ? 1.f / den[wi] : 1.f;
+  float rstd = dinv;
   if (w != nullptr) {
     float ss = 0.f;
-    for (int j = lane; j < dv; j += 32) ss = fmaf(row[j], row[j], ss);
+    for (int j = lane; j < dv; j += 32) {
+      const float v = row[j] * dinv;
+      ss = fmaf(v, v, ss);
+    }
     ss = warp_sum(ss);
-    rstd = 1.f / sqrtf(ss / (float)dv + eps);
+    rstd = dinv / sqrtf(ss / (float)dv + eps);
+    if (w_heads) w += (long long)h * dv;
   }
   for (int j = lane; j < dv; j += 32) {
     float v = row[j] * rstd;
@@ -512,6 +814,44 @@ static int pow2_at_least(int v) {
   return p;
 }
 
+// Generic scan: P lanes share a value column, each keeps at most 32 (16 for small heads) of its rows; more lanes where the columns would
+// leave warps idle.
+template <bool SC>
+static int launch_gla_scan(const float* qkv, long long ld, int q_off, int k_off, int v_off, const float* decay_in, long long lda,
+                           const float* decay_bias, float inv_tau, float q_scale, int S, int H, int dk, int dv, float* state, const int* cu,
+                           const int* slots, float* out, const MemoryGates& mg, cudaStream_t st) {
+  const int cols = dv + (SC ? 1 : 0);
+  int P = 1;
+  while ((dk + P - 1) / P > 32) P <<= 1;
+  while (P < 32 && (kRecThreads / 32) * (32 / P) / 2 >= cols && (dk + P - 1) / P > 4) P <<= 1;
+  const int KR = (dk + P - 1) / P;
+  const int CB = (kRecThreads / 32) * (32 / P);
+  const size_t smem = (size_t)(4 * kRecTok * dk + kRecTok * CB) * 4;
+  dim3 grid(S, H, (cols + CB - 1) / CB);
+  if (smem > 48 * 1024) {
+    SEQ_CUDA(cudaFuncSetAttribute(gla_scan_kernel<32, SC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    SEQ_CUDA(cudaFuncSetAttribute(gla_scan_kernel<16, SC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+  }
+  if (KR <= 16)
+    gla_scan_kernel<16, SC><<<grid, kRecThreads, smem, st>>>(qkv, ld, q_off, k_off, v_off, decay_in, lda, decay_bias, inv_tau, q_scale, H, dk, dv,
+                                                             P, state, cu, slots, out, mg);
+  else
+    gla_scan_kernel<32, SC><<<grid, kRecThreads, smem, st>>>(qkv, ld, q_off, k_off, v_off, decay_in, lda, decay_bias, inv_tau, q_scale, H, dk, dv,
+                                                             P, state, cu, slots, out, mg);
+  SEQ_LAUNCHED();
+  return KB2SEQ_OK;
+}
+
+template <int DK>
+static int launch_mlstm_reg(const float* qkv, long long ld, int q_off, int k_off, int v_off, float q_scale, int S, int H, int dv, float* state,
+                            const int* cu, const int* slots, float* out, const MemoryGates& mg, cudaStream_t st) {
+  const size_t smem = (size_t)(2 * 2 * kGlaTile * DK + 2 * kGlaTile * 34 + kGlaTile * kGlaWarps * 32) * 4;
+  if (smem > 48 * 1024) SEQ_CUDA(cudaFuncSetAttribute(mlstm_reg_kernel<DK>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+  mlstm_reg_kernel<DK><<<dim3(S, H, dv / 32 + 1), 32 * kGlaWarps, smem, st>>>(qkv, ld, q_off, k_off, v_off, q_scale, H, dv, state, cu, slots, out, mg);
+  SEQ_LAUNCHED();
+  return KB2SEQ_OK;
+}
+
 template <int DK>
 static int launch_gla_reg(const float* qkv, long long ld, int q_off, int k_off, int v_off, const float* alpha, float q_scale, int S, int H,
                           int dv, float* state, const int* cu, const int* slots, float* out, cudaStream_t st) {
@@ -547,24 +887,54 @@ KB2SEQ_API int kb2_seq_gla(const float* qkv, long long ld, int q_off, int k_off,
     if (dk == 128) return launch_gla_reg<128>(qkv, ld, q_off, k_off, v_off, scratch, q_scale, S, H, dv, state, cu, slots, out, st0);
     return launch_gla_reg<256>(qkv, ld, q_off, k_off, v_off, scratch, q_scale, S, H, dv, state, cu, slots, out, st0);
   }
-  // P lanes share a value column; each keeps at most 32 (16 for small heads) of its rows
-  int P = 1;
-  while ((dk + P - 1) / P > 32) P <<= 1;
-  const int KR = (dk + P - 1) / P;
-  const int CB = (kRecThreads / 32) * (32 / P);
-  const size_t smem = (size_t)(4 * kRecTok * dk + kRecTok * CB) * 4;
-  dim3 grid(S, H, (dv + CB - 1) / CB);
+  return launch_gla_scan<false>(qkv, ld, q_off, k_off, v_off, decay_in, lda, decay_bias, 1.f / tau, q_scale, S, H, dk, dv, state, cu, slots, out,
+                                MemoryGates{}, (cudaStream_t)stream);
+}
+
+KB2SEQ_API int kb2_seq_mlstm(const float* proj, long long ld, int q_off, int k_off, int v_off, int i_off, int f_off, const float* i_bias,
+                             const float* f_bias, float cap, float q_scale, int T, int S, int H, int dk, int dv, float* state, float* nstate,
+                             float* mstate, const int* cu, const int* slots, float* scratch, float* out, float* den, void* stream) {
+  if (!proj || !state || !nstate || !mstate || !cu || !slots || !scratch || !out || !den || T <= 0 || S <= 0 || H <= 0 || dk <= 0 || dv <= 0 ||
+      !(cap > 0.f))
+    return failf(KB2SEQ_ERR_VALUE, "mlstm: bad argument");
+  if (dk > 1024) return failf(KB2SEQ_ERR_VALUE, "mlstm: key size %d > 1024", dk);
+  if (H > 65535) return failf(KB2SEQ_ERR_VALUE, "mlstm: too many heads");
   cudaStream_t st = (cudaStream_t)stream;
-  if (smem > 48 * 1024) {
-    SEQ_CUDA(cudaFuncSetAttribute(gla_scan_kernel<32>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-    SEQ_CUDA(cudaFuncSetAttribute(gla_scan_kernel<16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+  float* keep = scratch;
+  float* add = keep + (long long)T * H;
+  float* mx = add + (long long)T * H;
+  const int threads = T >= kGateThreads ? kGateThreads : (T + 31) / 32 * 32;
+  mlstm_gates_kernel<<<dim3(S, H), threads, 0, st>>>(proj, ld, i_off, f_off, i_bias, f_bias, cap, H, mstate, cu, slots, keep, add, mx);
+  SEQ_LAUNCHED();
+  const MemoryGates mg{keep, add, mx, nstate, den};
+  const bool aligned = ((uintptr_t)proj & 15) == 0 && (ld & 3) == 0 && (q_off & 3) == 0 && (k_off & 3) == 0 && (v_off & 3) == 0;
+  if (aligned && (dk == 32 || dk == 64 || dk == 128 || dk == 256) && dv % 32 == 0 && dv / 32 < 65535) {
+#define KB2_MEM(DKV) launch_mlstm_reg<DKV>(proj, ld, q_off, k_off, v_off, q_scale, S, H, dv, state, cu, slots, out, mg, st)
+    if (dk == 32) return KB2_MEM(32);
+    if (dk == 64) return KB2_MEM(64);
+    if (dk == 128) return KB2_MEM(128);
+    return KB2_MEM(256);
+#undef KB2_MEM
   }
-  if (KR <= 16)
-    gla_scan_kernel<16><<<grid, kRecThreads, smem, st>>>(qkv, ld, q_off, k_off, v_off, decay_in, lda, decay_bias, 1.f / tau, q_scale, H, dk, dv,
-                                                         P, state, cu, slots, out);
-  else
-    gla_scan_kernel<32><<<grid, kRecThreads, smem, st>>>(qkv, ld, q_off, k_off, v_off, decay_in, lda, decay_bias, 1.f / tau, q_scale, H, dk, dv,
-                                                         P, state, cu, slots, out);
+  return launch_gla_scan<true>(proj, ld, q_off, k_off, v_off, nullptr, 0, nullptr, 1.f, q_scale, S, H, dk, dv, state, cu, slots, out, mg, st);
+}
+
+KB2SEQ_API int kb2_seq_rglru(const float* u, long long ldu, const float* z, long long ldz, long long zb, const float* y, long long ldy,
+                             const float* r_bias, const float* i_bias, const float* y_bias, const float* lam, int T, int S, int C, int bs,
+                             float* state, const int* cu, const int* slots, void* out, int dt_out, void* stream) {
+  if (!u || !z || !y || !lam || !state || !cu || !slots || !out || T <= 0 || S <= 0 || C <= 0 || bs <= 0 || C % bs || bad_dt(dt_out))
+    return failf(KB2SEQ_ERR_VALUE, "rglru: bad argument");
+  if ((C + 31) / 32 > 65535) return failf(KB2SEQ_ERR_VALUE, "rglru: too many channels");
+  rglru_scan_kernel<<<dim3(S, (C + 31) / 32), 32 * kRgWarps, 0, (cudaStream_t)stream>>>(u, ldu, z, ldz, zb, y, ldy, r_bias, i_bias, y_bias, lam, C, bs,
+                                                                                       state, cu, slots, out, dt_out);
+  SEQ_LAUNCHED();
+  return KB2SEQ_OK;
+}
+
+KB2SEQ_API int kb2_seq_split_blocks(const float* u, long long ldu, int T, int T_pad, int blocks, int bs, void* out, void* stream) {
+  if (!u || !out || T <= 0 || T_pad < T || blocks <= 0 || bs <= 0 || (bs & 1)) return failf(KB2SEQ_ERR_VALUE, "split_blocks: bad argument");
+  const long long n = (long long)T * blocks * (bs / 2);
+  split_blocks_kernel<<<(unsigned)((n + 255) / 256), 256, 0, (cudaStream_t)stream>>>(u, ldu, T, T_pad, blocks, bs, (bf16*)out);
   SEQ_LAUNCHED();
   return KB2SEQ_OK;
 }
@@ -594,11 +964,12 @@ KB2SEQ_API int kb2_seq_selective_scan(const float* x, long long ldx, const float
 }
 
 KB2SEQ_API int kb2_seq_head_norm_gate(const float* o, long long ldo, const float* w, float eps, const float* gate, long long ldg, int gate_act,
-                                      int T, int H, int dv, void* out, int dt_out, void* stream) {
+                                      int T, int H, int dv, void* out, int dt_out, const float* den, int w_heads, void* stream) {
   if (!o || !out || T <= 0 || H <= 0 || dv <= 0 || bad_dt(dt_out) || gate_act < 0 || gate_act > 1)
     return failf(KB2SEQ_ERR_VALUE, "head_norm_gate: bad argument");
   const long long nw = (long long)T * H;
-  head_norm_gate_kernel<<<(unsigned)((nw + 7) / 8), 256, 0, (cudaStream_t)stream>>>(o, ldo, w, eps, gate, ldg, gate_act, H, dv, T, out, dt_out);
+  head_norm_gate_kernel<<<(unsigned)((nw + 7) / 8), 256, 0, (cudaStream_t)stream>>>(o, ldo, w, eps, gate, ldg, gate_act, H, dv, T, out, dt_out, den,
+                                                                                      w_heads);
   SEQ_LAUNCHED();
   return KB2SEQ_OK;
 }

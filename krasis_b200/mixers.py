@@ -17,20 +17,26 @@ libkrasis_b200_seq (`krasis_b200.seqops`): a model composes them (krasis_b200/vo
                           of q and of k, rotation of dimension i with i + dims / 2, a frequency table of the caller, tanh soft-capped
                           scores, a softmax sink per head, mean-pooled blocks of keys and values before the window, values cached
                           rotated by their positions with the output turned back, an output gate per element, query and key norms
-                          without weights, a penalty per head that grows with the distance to the key)
+                          without weights, a penalty per head that grows with the distance to the key, an amplitude on sin and cos,
+                          values that are the projected keys, one added to the softmax denominator)
   GatedLinearAttention    S <- diag(alpha) S + k v^T with one decay per key channel, alpha = sigmoid(.)^(1 / tau) from a low-rank
                           projection; per-head RMS norm of the read-out with a SiLU gate
   SelectiveScan           Mamba: input / gate projection, short causal convolution, input-dependent step sizes and B / C, diagonal
                           state per channel in fp32 slots
-  SideBySide              two mixers that read the same input: each output RMS-normed over the width, then averaged
+  MatrixMemory            mLSTM: S <- keep S + add k v^T with exponential gates relative to a running maximum, a key sum as normaliser;
+                          state, key sum and maximum in fp32 slots; unit RMS norm per head, a sigmoid gate per element
+  GatedRecurrentUnit      Griffin's recurrent block: a convolved branch through a diagonal recurrence with block-diagonal gates (real-gated
+                          linear recurrent unit), times a tanh-GELU branch; state per channel in fp32 slots
+  SideBySide              two mixers that read the same input: each output RMS-normed over the width, then averaged; or their sum with
+                          fixed factors
   ChannelDeltaMixer       the gated delta rule with one decay per head and key channel (low-rank decay and output-gate projections,
                           sigmoid output gate)
   GatedMLP                down(act(gate h) * (up h)): tanh-GELU, SiLU, or the clamped swish form g' sigmoid(a g') (u' + 1); without a
-                          gate: down(relu(up h)^2)
+                          gate: down(relu(up h)^2); optional biases
   RoutedExperts           softmax / sigmoid router with a choice correction, expert groups (scored by their best or their two best
                           outputs) and identity experts, or a choice by the biased logits with a softmax over the chosen ones; top-k
                           experts of any of those forms (binned tile GEMMs; a GEMV form for steps of few tokens) plus an optional shared
-                          expert with an optional per-token sigmoid gate
+                          expert with an optional per-token sigmoid gate; the weight multiplies an expert's output or its input
   TokenSideInput          per-layer token table slice, gated by a projection of the residual stream, RMS-normed
 `lin(a, w, out_dtype)` picks the GEMM: the tcgen05 kernel of the core library for large aligned bf16 products, the generic
 kernel of the sequence library otherwise (any shape, fp32 or bf16).
@@ -340,7 +346,7 @@ class SelectiveScan:
     def forward(self, h: torch.Tensor, tb: ops.StepTables, tail: torch.Tensor, state: torch.Tensor) -> torch.Tensor:
         lib, T = ops.load(), h.shape[0]
         proj = lin(h, self.w_in, torch.float32)                                               # [T, x: C | z: C]
-        xc = ops.conv(proj, self.C, self.taps, self.conv_b, True, tail, tb, bias_after=True)  # [T, C] fp32
+        xc = ops.conv(proj, self.C, self.taps, None, True, tail, tb, bias_out=self.conv_b)    # [T, C] fp32
         big = self.dtype == torch.bfloat16 and T >= 256 and bool(_core_lib())
         xp = lin(xc.to(torch.bfloat16) if big else xc, self.w_x, torch.float32, min_n=16)     # [T, dt: R | B: N | C: N]
         dt_in = lin_cols(xp, 0, self.R, self.w_dt, self.dtype)                                # [T, C]
@@ -353,11 +359,136 @@ class SelectiveScan:
         return lin(y, self.w_o, torch.float32)
 
 
-class SideBySide:
-    """Two mixers read the same input; the result is coef (left / rms(left) * w_left + right / rms(right) * w_right) over the width."""
+class MatrixMemory:
+    """weights: q, k [H dk, W], v, g [H dv, W], i, f [H, W], i_b, f_b [H], norm [H dv], o [W, H dv].
 
-    def __init__(self, left, right, w_left: torch.Tensor, w_right: torch.Tensor, eps: float, device, coef: float = 0.5):
+    Per head: log gates i = cap tanh((i h + i_b) / cap) and f = logsigmoid(cap tanh((f h + f_b) / cap)); running maximum
+    m_t = max(f + m_(t-1), i) from m_0 = 0; S <- exp(f + m_(t-1) - m_t) S + exp(i - m_t) k v^T and the key sum n likewise;
+    o = S^T q / (max(|n . q|, exp(-m_t)) + 1e-6) with q = (q h) dk^-1/2; out = o / rms(o) per head, times norm, times sigmoid(g h), then the
+    output projection (the matrix memory of Beck et al., "xLSTM: Extended Long Short-Term Memory").  S [slots, H, dk, dv], n [slots, H, dk]
+    and m [slots, H] are fp32; the gates are evaluated in fp64."""
+
+    def __init__(self, weights: dict, heads: int, dim: int, vdim: int, gate_cap: float, eps: float, dtype, device):
+        self.H, self.dk, self.dv, self.cap = heads, dim, vdim, float(gate_cap)
+        self.eps, self.dtype, self.device = float(eps), dtype, device
+        d = lambda t: t.to(device=device, dtype=dtype).contiguous()
+        f = lambda t: t.to(device=device, dtype=torch.float32).contiguous()
+        names = ("q", "k", "v", "g", "i", "f")
+        rows = [weights[k] for k in names]
+        offs, at = {}, 0
+        for k, r in zip(names, rows):
+            offs[k], at = at, at + r.shape[0]
+        self.q_off, self.k_off, self.v_off, self.g_off, self.i_off, self.f_off = (offs[k] for k in names)
+        if at % 16:                                                                           # a width the tensor-core product takes
+            rows.append(torch.zeros(-at % 16, rows[0].shape[1], dtype=rows[0].dtype))
+        self.w_in = d(torch.cat(rows, 0))                                                     # one projection of the layer input
+        self.i_b = f(weights["i_b"]) if "i_b" in weights else None
+        self.f_b = f(weights["f_b"]) if "f_b" in weights else None
+        self.norm, self.w_o = f(weights["norm"]), d(weights["o"])
+        if weights["q"].shape[0] != heads * dim or weights["v"].shape[0] != heads * vdim or weights["i"].shape[0] != heads or self.norm.numel() != heads * vdim:
+            raise ValueError("matrix memory: tensor shapes do not match heads x dim / vdim")
+
+    def register_state(self, pool):
+        """(S [slots, H, dk, dv], n [slots, H, dk], m [slots, H]) in a RecurrentStatePool."""
+        return pool.register(self.H, self.dk, self.dv), pool.register(self.H, self.dk), pool.register(self.H)
+
+    def forward(self, h: torch.Tensor, tb: ops.StepTables, state: torch.Tensor, nstate: torch.Tensor, mstate: torch.Tensor) -> torch.Tensor:
+        lib, T, H = ops.load(), h.shape[0], self.H
+        proj = lin(h, self.w_in, torch.float32)
+        o = torch.empty((T, H * self.dv), dtype=torch.float32, device=h.device)
+        small = torch.empty((4, T, H), dtype=torch.float32, device=h.device)                  # keep, add, maximum | divisor
+        ops.check(lib.kb2_seq_mlstm(proj.data_ptr(), proj.stride(0), self.q_off, self.k_off, self.v_off, self.i_off, self.f_off, ops._ptr(self.i_b),
+                                    ops._ptr(self.f_b), self.cap, float(self.dk) ** -0.5, T, tb.S, H, self.dk, self.dv, state.data_ptr(),
+                                    nstate.data_ptr(), mstate.data_ptr(), tb.cu.data_ptr(), tb.slots.data_ptr(), small.data_ptr(), o.data_ptr(),
+                                    small[3].data_ptr(), torch.cuda.current_stream(h.device).cuda_stream))
+        o = ops.head_norm_gate(o, H, self.dv, self.dtype, norm=self.norm, eps=self.eps, gate=proj[:, self.g_off:], gate_act="sigmoid", den=small[3])
+        return lin(o, self.w_o, torch.float32)
+
+
+class GatedRecurrentUnit:
+    """weights: x, y [C, W], x_b, y_b [C], conv [C, taps], conv_b [C], ra, ri [blocks, C / blocks, C / blocks], ra_b, ri_b [blocks, C / blocks],
+    lam [C], o [W, C].
+
+    u = conv(x h + x_b) + conv_b; per block r = sigmoid(ra u + ra_b), i = sigmoid(ri u + ri_b); log a = -8 r softplus(lam);
+    S <- a S + sqrt(1 - a^2) i u; out = o (S gelu_tanh(y h + y_b)) (the recurrent block of De et al., "Griffin: Mixing Gated Linear
+    Recurrences with Local Attention for Efficient Language Models").  The state [slots, C], the convolution's last taps - 1 inputs, the
+    gates with their products and the decays are fp32."""
+
+    def __init__(self, weights: dict, width: int, blocks: int, taps: int, dtype, device):
+        self.C, self.B, self.K = int(width), int(blocks), int(taps)
+        if self.C % self.B:
+            raise ValueError("the blocks must divide the width of the recurrence")
+        self.bs, self.dtype, self.device = self.C // self.B, dtype, device
+        d = lambda t: t.to(device=device, dtype=dtype).contiguous()
+        f = lambda t: t.to(device=device, dtype=torch.float32).contiguous()
+        rows = [weights["x"], weights["y"]]                                                   # the convolution reads the first C columns
+        pad = -2 * self.C % 16
+        if pad:
+            rows.append(torch.zeros(pad, rows[0].shape[1], dtype=rows[0].dtype))
+        self.w_in, self.w_o = d(torch.cat(rows, 0)), d(weights["o"])
+        opt = lambda k: f(weights[k]).reshape(-1) if k in weights else None
+        self.x_b, self.y_b, self.conv_b, self.ra_b, self.ri_b = (opt(k) for k in ("x_b", "y_b", "conv_b", "ra_b", "ri_b"))
+        self.taps, self.lam = f(weights["conv"]), f(weights["lam"])
+        self.w_gates = d(torch.cat([weights["ra"], weights["ri"]], 1))                        # [blocks, 2 bs, bs]: both gates of a block
+        if self.taps.shape != (self.C, self.K) or self.w_gates.shape != (self.B, 2 * self.bs, self.bs) or self.lam.numel() != self.C:
+            raise ValueError("recurrent unit: tensor shapes do not match width / blocks / taps")
+        # long bfloat16 steps: the gate products of a block run on the tensor cores with the fp32 inputs as a high and a low bfloat16 part
+        self.tc_min_tokens = 256
+        self.w_gates_twice = torch.cat([self.w_gates, self.w_gates], 2).contiguous() if dtype == torch.bfloat16 and self.bs % 32 == 0 else None
+        self._tiles = {}
+
+    def register_state(self, pool):
+        """(conv tail [slots, C, taps - 1], state [slots, C]) in a RecurrentStatePool."""
+        return pool.register(self.C, max(self.K - 1, 1)), pool.register(self.C)
+
+    def _gate_products(self, u: torch.Tensor):
+        """u [T, C] fp32 -> (products, row stride, block stride) with both gates of a channel bs columns apart."""
+        T, dev = u.shape[0], u.device
+        s = torch.cuda.current_stream(dev).cuda_stream
+        core = _core_lib() if self.w_gates_twice is not None and T >= self.tc_min_tokens else False
+        if not core:
+            z = torch.empty((T, self.B, 2 * self.bs), dtype=torch.float32, device=dev)
+            ops.gemm_heads(u.view(T, self.B, self.bs), self.w_gates, z)
+            return z, 2 * self.C, 2 * self.bs
+        from . import capi
+        tp = (T + 127) // 128 * 128
+        if tp not in self._tiles:                              # row tile -> block, and the number of row tiles
+            self._tiles[tp] = (torch.arange(self.B, dtype=torch.int32, device=dev).repeat_interleave(tp // 128).contiguous(),
+                               torch.tensor([self.B * (tp // 128)], dtype=torch.int32, device=dev))
+        tile_block, n_tiles = self._tiles[tp]
+        parts = torch.empty((self.B * tp, 2 * self.bs), dtype=torch.bfloat16, device=dev)
+        ops.check(ops.load().kb2_seq_split_blocks(u.data_ptr(), u.stride(0), T, tp, self.B, self.bs, parts.data_ptr(), s))
+        z = torch.empty((self.B * tp, 2 * self.bs), dtype=torch.float32, device=dev)
+        capi.check(core.kb2_linear_bf16_grouped(parts.data_ptr(), self.w_gates_twice.data_ptr(), z.data_ptr(), self.B * tp, 2 * self.bs, 2 * self.bs, 1,
+                                                tile_block.data_ptr(), n_tiles.data_ptr(), self.B, dev.index or 0, s))
+        return z, 2 * self.bs, tp * 2 * self.bs
+
+    def forward(self, h: torch.Tensor, tb: ops.StepTables, tail: torch.Tensor, state: torch.Tensor) -> torch.Tensor:
+        T = h.shape[0]
+        proj = lin(h, self.w_in, torch.float32)                                               # [T, x: C | y: C]
+        u = ops.conv(proj, self.C, self.taps, self.x_b, False, tail, tb, bias_out=self.conv_b)
+        z, ldz, zb = self._gate_products(u)
+        o = torch.empty((T, self.C), dtype=self.dtype, device=h.device)
+        ops.check(ops.load().kb2_seq_rglru(u.data_ptr(), u.stride(0), z.data_ptr(), ldz, zb, proj[:, self.C:].data_ptr(), proj.stride(0),
+                                           ops._ptr(self.ra_b), ops._ptr(self.ri_b), ops._ptr(self.y_b), self.lam.data_ptr(), T, tb.S, self.C,
+                                           self.bs, state.data_ptr(), tb.cu.data_ptr(), tb.slots.data_ptr(), o.data_ptr(), ops.dt_code(self.dtype),
+                                           torch.cuda.current_stream(h.device).cuda_stream))
+        return lin(o, self.w_o, torch.float32)
+
+
+class SideBySide:
+    """Two mixers read the same input; the result is coef (left / rms(left) * w_left + right / rms(right) * w_right) over the width.
+    Without norm weights (scales = (a, b)): a left + b right; the two terms go to the residual update as they are (`scales`,
+    ops.residual_post_rms), no pass of their own."""
+
+    def __init__(self, left, right, w_left: torch.Tensor = None, w_right: torch.Tensor = None, eps: float = 0.0, device=None, coef: float = 0.5,
+                 scales=None):
         self.left, self.right, self.eps, self.coef = left, right, float(eps), float(coef)
+        self.scales = (float(scales[0]), float(scales[1])) if scales is not None else None
+        if (self.scales is None) == (w_left is None or w_right is None):
+            raise ValueError("norm weights for both sides, or a scale for each")
+        if self.scales is not None:
+            return
         self.w_left = w_left.to(device=device, dtype=torch.float32).contiguous()
         self.w_right = w_right.to(device=device, dtype=torch.float32).contiguous()
 
@@ -430,7 +561,8 @@ class ChannelDeltaMixer:
 class GatedMLP:
     """weights: gate, up [F, W], down [W, F].  act: "gelu_tanh" (gelu(g) u), "silu" (silu(g) u) or "clamped_swish"
     (g' sigmoid(alpha g') (u' + 1) with g' = min(g, limit), u' = clamp(u, -limit, limit)).  gated False: weights up, down only and
-    down(act(up h)) with act "relu2" (the square of relu)."""
+    down(act(up h)) with act "relu2" (the square of relu).  Optional biases gate_b, up_b [F] (inside the activation pass) and down_b [W]:
+    down_b is not part of `forward`'s result, the residual update adds it (`out_bias`, ops.residual_post_rms)."""
 
     KINDS = {"gelu_tanh": ops.GLU_GELU_TANH, "silu": ops.GLU_SILU, "clamped_swish": ops.GLU_CLAMPED_SWISH, "relu2": ops.ACT_RELU2}
 
@@ -441,10 +573,19 @@ class GatedMLP:
         self.w_gu = d(torch.cat([weights["gate"], weights["up"]], 0)) if gated else d(weights["up"])
         self.w_down, self.dtype = d(weights["down"]), dtype
         self.kind, self.limit, self.alpha = self.KINDS[act], float(limit), float(alpha)
+        f = lambda t: t.to(device=device, dtype=torch.float32).contiguous()
+        names = ("gate_b", "up_b") if gated else ("up_b",)
+        self.bias = None
+        if any(n in weights for n in names):
+            self.bias = f(torch.cat([weights[n].float() if n in weights else torch.zeros(self.w_down.shape[1]) for n in names], 0))
+        self.out_bias = f(weights["down_b"]) if "down_b" in weights else None
 
     def forward(self, h: torch.Tensor) -> torch.Tensor:
         gu = lin(h, self.w_gu, self.dtype)
-        a = ops.act_mul(gu, self.dtype) if self.kind == ops.GLU_GELU_TANH else ops.glu(gu, self.dtype, self.kind, self.limit, self.alpha)
+        if self.kind == ops.GLU_GELU_TANH and self.bias is None:
+            a = ops.act_mul(gu, self.dtype)
+        else:
+            a = ops.glu(gu, self.dtype, self.kind, self.limit, self.alpha, bias=self.bias)
         return lin(a, self.w_down, torch.float32)
 
 
@@ -499,13 +640,17 @@ class MultiMapAttention:
     the pair layout of the keys) and each head's output is turned back by the query's position, ahead of the gate.
     gate_per_element: g is [H dv, W], one sigmoid gate per output element (default [H, W]: one per head).
     qk_unit: every query and key vector is divided by its root mean square, without a weight.
-    slopes [H]: slopes[h] times the distance (query position - key position) is taken off head h's scores, after scale and cap."""
+    slopes [H]: slopes[h] times the distance (query position - key position) is taken off head h's scores, after scale and cap.
+    rot_amp: sin and cos of the query / key rotation are multiplied by it.  keys_as_values: no v tensor, the values are the keys as
+    projected, ahead of norm and rotation (dim == vdim, one map).  off_by_one: the softmax denominator of every head is 1 + sum exp(s)
+    (a sink of score 0)."""
 
     def __init__(self, weights: dict, heads: int, kv_heads: int, maps: int, dim: int, vdim: int, scale: float, eps: float, dtype, device,
                  chunk=None, window=None, rot_dims: int = 0, rot_base: float = 10000.0, rot_factor: float = 1.0, map_coef=None,
                  unit_norm: bool = False, post_scale: float = 1.0, own_kv: bool = True, conv_taps: int = 0, norm_whole: bool = False,
                  rot_half: bool = False, rot_freq=None, softcap: float = 0.0, pool: int = 0, rot_values: bool = False,
-                 gate_per_element: bool = False, qk_unit: bool = False, slopes=None):
+                 gate_per_element: bool = False, qk_unit: bool = False, slopes=None, rot_amp: float = 1.0, keys_as_values: bool = False,
+                 off_by_one: bool = False):
         if heads % kv_heads:
             raise ValueError("heads must be a multiple of kv_heads")
         if rot_dims > dim or rot_dims % 2:
@@ -533,12 +678,19 @@ class MultiMapAttention:
         d = lambda t: t.to(device=device, dtype=dtype).contiguous()
         f = lambda t: t.to(device=device, dtype=torch.float32).contiguous()
         self.sink = f(weights["sink"]) if "sink" in weights else None
+        if off_by_one:
+            if self.sink is not None:
+                raise ValueError("a sink of score 0, or one per head")
+            self.sink = torch.zeros(heads, dtype=torch.float32, device=device)
         if self.sink is not None and self.sink.numel() != heads:
             raise ValueError("one sink per head")
+        self.rot_amp, self.kv_one = float(rot_amp), bool(keys_as_values)
+        if self.kv_one and (dim != vdim or self.M != 1 or not own_kv or "v" in weights):
+            raise ValueError("keys as values: one map, dim == vdim, projections of the layer's own and no v tensor")
         self.map_coef = f(torch.as_tensor(map_coef, dtype=torch.float64)) if map_coef is not None else None
         if self.map_coef is not None and self.map_coef.numel() != self.M:
             raise ValueError("one coefficient per map")
-        names = ["q"] + (["k", "v"] if own_kv else [])
+        names = ["q"] + ((["k"] if self.kv_one else ["k", "v"]) if own_kv else [])
         rows = [weights[n] for n in names]
         self.gate_off = sum(r.shape[0] for r in rows) if "g" in weights else -1
         if "g" in weights:
@@ -634,7 +786,8 @@ class MultiMapAttention:
         ops.check(lib.kb2_seq_head_kv_prep(proj.data_ptr(), ldp, T, H, G if self.own_kv else 0, M, self.d, self.dv, ops._ptr(bias),
                                            ops._ptr(self.q_norm), ops._ptr(self.k_norm), self.eps, ops._ptr(self.freq), self.rot_dims,
                                            tb.positions.data_ptr(), tb.seq_of.data_ptr(), tb.pages.data_ptr(), tb.max_pages, page_size,
-                                           kc.data_ptr(), vc.data_ptr(), dtc, int(self.norm_whole), int(self.rot_half), ops._ptr(self.vfreq), s))
+                                           kc.data_ptr(), vc.data_ptr(), dtc, int(self.norm_whole), int(self.rot_half), ops._ptr(self.vfreq),
+                                           self.rot_amp, int(self.kv_one), s))
         if self.pool:                                # the tokens that complete a block write its mean key and value
             ops.check(lib.kb2_seq_kv_pool(kc.data_ptr(), vc.data_ptr(), kp.data_ptr(), vp.data_ptr(), dtc, G * M * self.d, G * self.dv, self.pool,
                                           T, tb.positions.data_ptr(), tb.seq_of.data_ptr(), tb.pages.data_ptr(), tb.max_pages, page_size, s))
@@ -693,17 +846,23 @@ class RoutedExperts:
     Scores are softmax (or sigmoid) of the fp32 router logits over all E + identity outputs; the choice adds `correction`; the outputs
     form `groups` equal groups of neighbours of which the `keep` with the largest group score stay eligible (group_score "max": the
     group's largest choice, "top2": the sum of its two largest); the `top` largest choices are taken and weighted by their scores
-    (divided by their sum if `renorm`, times out_scale).  The last `identity` outputs are identity experts: they return their input."""
+    (divided by their sum if `renorm`, times out_scale).  The last `identity` outputs are identity experts: they return their input.
+
+    weight_input: the weight multiplies the expert's input, out = sum expert(w h).  Gate and up products are linear in it, so the weight
+    joins the activation pass (gated experts, no identity experts)."""
 
     def __init__(self, weights: dict, experts: int, identity: int, top: int, dtype, device, groups: int = 1, keep: int = 1,
                  score: str = "softmax", renorm: bool = False, out_scale: float = 1.0, gated: bool = True, act: str = "silu",
-                 group_score: str = "max", limit: float = 0.0, alpha: float = 1.0, shared_limit=None):
+                 group_score: str = "max", limit: float = 0.0, alpha: float = 1.0, shared_limit=None, weight_input: bool = False):
         d = lambda t: t.to(device=device, dtype=dtype).contiguous()
         self.E, self.ident, self.top, self.groups, self.keep = int(experts), int(identity), int(top), int(groups), int(keep)
         self.score, self.renorm, self.out_scale, self.dtype, self.device = score, bool(renorm), float(out_scale), dtype, device
         self.gated, self.group_score = bool(gated), group_score
         if gated == (act == "relu2") or act not in ("silu", "clamped_swish", "relu2") or group_score not in ("max", "top2"):
             raise ValueError("experts: silu or clamped_swish with a gate or relu2 without; group_score max or top2")
+        self.weight_input = bool(weight_input)
+        if self.weight_input and self.ident:
+            raise ValueError("weights on the experts' inputs: no identity experts")
         if score not in ops.ROUTE_SCORES:
             raise ValueError(f"router score {score!r}")
         self.act_kind, self.limit, self.alpha = GatedMLP.KINDS[act], float(limit), float(alpha)
@@ -756,7 +915,7 @@ class RoutedExperts:
         return (self.dtype == torch.bfloat16 and h.dtype == torch.bfloat16 and h.is_contiguous() and W % 64 == 0 and self.F % 64 == 0
                 and slots >= self.tc_min_rows_per_expert * self.E and bool(_core_lib()))
 
-    def _forward_tensor_core(self, h, ids, slots):
+    def _forward_tensor_core(self, h, ids, slots, in_w):
         """Long bfloat16 steps: rows gathered into the binned order (runs padded to the 128-row tiles of the tcgen05 GEMM), then ONE
         grouped GEMM per projection: every row tile multiplies its expert's matrix, picked from the device-side tile table, and only
         the tiles that exist are computed — no host round trip."""
@@ -771,7 +930,8 @@ class RoutedExperts:
         gu = torch.empty((rows, F1), dtype=torch.bfloat16, device=dev)
         capi.check(core.kb2_linear_bf16_grouped(xs.data_ptr(), self.w_gu.data_ptr(), gu.data_ptr(), rows, F1, W, 0, t["tile_expert"].data_ptr(),
                                                 t["n_tiles"].data_ptr(), E, di, s))
-        act = ops.glu(gu, torch.bfloat16, self.act_kind, self.limit, self.alpha, n_tiles=t["n_tiles"], tile_rows=128)
+        act = ops.glu(gu, torch.bfloat16, self.act_kind, self.limit, self.alpha, n_tiles=t["n_tiles"], tile_rows=128, row_w=in_w,
+                      row_map=t["slot_row"])
         y = torch.empty((rows, W), dtype=torch.float32, device=dev)
         capi.check(core.kb2_linear_bf16_grouped(act.data_ptr(), self.w_down.data_ptr(), y.data_ptr(), rows, W, F, 1, t["tile_expert"].data_ptr(),
                                                 t["n_tiles"].data_ptr(), E, di, s))
@@ -789,18 +949,19 @@ class RoutedExperts:
         ids, wts, z = self.route(h)
         dt, dtc = self.dtype, ops.dt_code(self.dtype)
         slots = T * top
+        in_w, out_w = (wts, None) if self.weight_input else (None, wts)       # where the weights go: into the activation pass or the sum
         y = pos = None
         if E and T <= self.gemv_max_tokens:
             F2 = self.w_gu.shape[1]
             gu = torch.empty((slots, F2), dtype=dt, device=dev)
             ops.check(lib.kb2_seq_moe_gemv(h.data_ptr(), ops.dt_code(h.dtype), h.stride(0), top, ids.data_ptr(), E, self.w_gu.data_ptr(), dtc, W,
                                            F2 * W, gu.data_ptr(), dtc, F2, slots, F2, W, s))
-            act = ops.glu(gu, dt, self.act_kind, self.limit, self.alpha)
+            act = ops.glu(gu, dt, self.act_kind, self.limit, self.alpha, row_w=in_w)
             y = torch.empty((slots, W), dtype=torch.float32, device=dev)
             ops.check(lib.kb2_seq_moe_gemv(act.data_ptr(), dtc, self.F, 1, ids.data_ptr(), E, self.w_down.data_ptr(), dtc, self.F, W * self.F,
                                            y.data_ptr(), 0, W, slots, W, self.F, s))
         elif E and self._tensor_core_ok(h, slots):
-            y, pos = self._forward_tensor_core(h, ids, slots)
+            y, pos = self._forward_tensor_core(h, ids, slots, in_w)
         elif E:
             F2, tile = self.w_gu.shape[1], self.tile
             t = self._bin(ids, slots, tile)
@@ -808,14 +969,14 @@ class RoutedExperts:
             gu = torch.empty((max_rows, F2), dtype=dt, device=dev)
             ops.check(lib.kb2_seq_moe_gemm(h.data_ptr(), ops.dt_code(h.dtype), h.stride(0), slot_row.data_ptr(), top, self.w_gu.data_ptr(), dtc, W,
                                            F2 * W, gu.data_ptr(), dtc, F2, F2, W, tile_expert.data_ptr(), n_tiles.data_ptr(), max_tiles, tile, s))
-            act = ops.glu(gu, dt, self.act_kind, self.limit, self.alpha, n_tiles=n_tiles, tile_rows=tile)
+            act = ops.glu(gu, dt, self.act_kind, self.limit, self.alpha, n_tiles=n_tiles, tile_rows=tile, row_w=in_w, row_map=slot_row)
             y = torch.empty((max_rows, W), dtype=torch.float32, device=dev)
             ops.check(lib.kb2_seq_moe_gemm(act.data_ptr(), dtc, self.F, None, 1, self.w_down.data_ptr(), dtc, self.F, W * self.F, y.data_ptr(), 0,
                                            W, W, self.F, tile_expert.data_ptr(), n_tiles.data_ptr(), max_tiles, tile, s))
         shared = self.shared.forward(h) if self.shared is not None else None
         out = torch.empty((T, W), dtype=torch.float32, device=dev)
         sg = z[:, self.sg_col:] if (self.sg_col >= 0 and shared is not None) else None
-        ops.check(lib.kb2_seq_moe_combine(ops._ptr(y), ops._ptr(pos), ids.data_ptr(), wts.data_ptr(), T, top, E, self.ident, h.data_ptr(),
+        ops.check(lib.kb2_seq_moe_combine(ops._ptr(y), ops._ptr(pos), ids.data_ptr(), ops._ptr(out_w), T, top, E, self.ident, h.data_ptr(),
                                           ops.dt_code(h.dtype), ops._ptr(shared), out.data_ptr(), W, ops._ptr(sg), z.stride(0), s))
         return out
 

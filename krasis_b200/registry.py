@@ -52,6 +52,13 @@ def _kugalorn(model_dir, dtype=torch.bfloat16, device=0, **kw):
     return KugalornModel.from_pretrained(model_dir, dtype=dtype, device=device, **kw)
 
 
+def _kivurax(model_dir, dtype=torch.bfloat16, device=0, **kw):
+    from .build import build_seq
+    build_seq()
+    from .kivurax import KivuraxModel
+    return KivuraxModel.from_pretrained(model_dir, dtype=dtype, device=device, **kw)
+
+
 def _hf_moe(model_dir, dtype=torch.bfloat16, device=0, **kw):
     if dtype != torch.bfloat16:
         raise ValueError("the MoE prefill models run in bfloat16 only")
@@ -66,6 +73,7 @@ register("Megolorn", _megolorn)
 register("Gurozen", _gurozen)
 register("Zaronex", _zaronex)
 register("Kugalorn", _kugalorn)
+register("Kivurax", _kivurax)
 for _name in _HF_MOE:
     register(_name, _hf_moe)
 

@@ -25,17 +25,17 @@ SIGNATURES = {
     "kb2_seq_latent_window_attn": (_I, [_P, _P, _L, _I, _I, _I, _I, _I, _P, _P, _I, _P, _P, _P, _I, _I, _P, _F, _I, _P, _P, _I, _I, _P, _P, _P, _L, _P]),
     "kb2_seq_conv_silu": (_I, [_P, _L, _I, _I, _I, _I, _P, _P, _P, _P, _P, _P, _P]),
     "kb2_seq_delta_rule": (_I, [_P, _I, _P, _L, _I, _I, _I, _I, _I, _I, _I, _I, _I, _P, _P, _P, _F, _P, _P, _P, _P, _P, _I, _P]),
-    "kb2_seq_conv": (_I, [_P, _L, _I, _I, _I, _I, _P, _P, _I, _P, _P, _P, _P, _P, _P]),
+    "kb2_seq_conv": (_I, [_P, _L, _I, _I, _I, _I, _P, _P, _P, _I, _P, _P, _P, _P, _P, _P]),
     "kb2_seq_residual_scale_rms": (_I, [_P, _P, _F, _P, _F, _P, _I, _I, _I, _F, _P]),
     "kb2_seq_delta_rule_ch": (_I, [_P, _I, _P, _L, _P, _L, _P, _L, _I, _I, _I, _I, _I, _I, _I, _P, _P, _P, _F, _P, _P, _P, _P, _P, _I, _P]),
     "kb2_seq_residual_add_norm": (_I, [_P, _P, _P, _P, _P, _P, _I, _I, _I, _F, _P]),
-    "kb2_seq_head_kv_prep": (_I, [_P, _L, _I, _I, _I, _I, _I, _I, _P, _P, _P, _F, _P, _I, _P, _P, _P, _I, _I, _P, _P, _I, _I, _I, _P, _P]),
+    "kb2_seq_head_kv_prep": (_I, [_P, _L, _I, _I, _I, _I, _I, _I, _P, _P, _P, _F, _P, _I, _P, _P, _P, _I, _I, _P, _P, _I, _I, _I, _P, _F, _I, _P]),
     "kb2_seq_kv_pool": (_I, [_P, _P, _P, _P, _I, _I, _I, _I, _I, _P, _P, _P, _I, _I, _P]),
     "kb2_seq_paged_attn": (_I, [_P, _L, _I, _I, _I, _I, _I, _I, _P, _P, _I, _P, _P, _P, _I, _I, _F, _I, _I, _P, _I, _P, _P, _P, _I, _F, _P, _I,
                                 _P, _P, _I, _P, _P]),
     "kb2_seq_pool_merge": (_I, [_P, _P, _P, _P, _I, _I, _I, _P, _P, _I, _P]),
     "kb2_seq_attn_finish": (_I, [_P, _P, _P, _I, _I, _I, _I, _I, _P, _I, _F, _F, _P, _L, _P, _I, _P, _P, _I, _I, _P, _P, _I, _P]),
-    "kb2_seq_glu": (_I, [_P, _I, _L, _P, _I, _L, _I, _I, _F, _F, _P, _I, _P]),
+    "kb2_seq_glu": (_I, [_P, _I, _L, _P, _I, _L, _I, _I, _F, _F, _P, _I, _P, _P, _P, _P]),
     "kb2_seq_route": (_I, [_P, _L, _I, _I, _P, _I, _I, _I, _I, _I, _F, _P, _P, _I, _P, _P]),
     "kb2_seq_moe_tile_rows": (_I, []),
     "kb2_seq_moe_bin": (_I, [_P, _L, _I, _I, _P, _P, _P, _P, _P, _P, _L, _P, _P]),
@@ -44,7 +44,11 @@ SIGNATURES = {
     "kb2_seq_moe_combine": (_I, [_P, _P, _P, _P, _I, _I, _I, _I, _P, _I, _P, _P, _I, _P, _L, _P]),
     "kb2_seq_gla": (_I, [_P, _L, _I, _I, _I, _P, _L, _P, _F, _F, _I, _I, _I, _I, _I, _P, _P, _P, _P, _P, _P]),
     "kb2_seq_selective_scan": (_I, [_P, _L, _P, _L, _P, _P, _L, _I, _P, _L, _I, _P, _P, _I, _I, _I, _I, _P, _P, _P, _P, _I, _P]),
-    "kb2_seq_head_norm_gate": (_I, [_P, _L, _P, _F, _P, _L, _I, _I, _I, _I, _P, _I, _P]),
+    "kb2_seq_head_norm_gate": (_I, [_P, _L, _P, _F, _P, _L, _I, _I, _I, _I, _P, _I, _P, _I, _P]),
+    "kb2_seq_mlstm": (_I, [_P, _L, _I, _I, _I, _I, _I, _P, _P, _F, _F, _I, _I, _I, _I, _I, _P, _P, _P, _P, _P, _P, _P, _P, _P]),
+    "kb2_seq_rglru": (_I, [_P, _L, _P, _L, _L, _P, _L, _P, _P, _P, _P, _I, _I, _I, _I, _P, _P, _P, _P, _I, _P]),
+    "kb2_seq_split_blocks": (_I, [_P, _L, _I, _I, _I, _I, _P, _P]),
+    "kb2_seq_residual_post_rms": (_I, [_P, _P, _F, _P, _F, _P, _F, _P, _P, _P, _I, _I, _I, _F, _P]),
     "kb2_seq_rms_rows": (_I, [_P, _L, _I, _P, _F, _P, _I, _L, _I, _P]),
     "kb2_seq_branch_merge": (_I, [_P, _P, _P, _P, _F, _F, _P, _I, _I, _P]),
     "kb2_seq_depth_mix": (_I, [_P, _L, _I, _P, _P, _P, _P, _P, _I, _I, _I, _F, _P]),
@@ -252,13 +256,17 @@ def residual_add_norm(x, y=None, y2=None, out_norm=None, out_dtype=torch.float32
 GLU_GELU_TANH, GLU_SILU, GLU_CLAMPED_SWISH, ACT_RELU2 = 0, 1, 2, 3
 
 
-def glu(gate_up: torch.Tensor, out_dtype, kind: int, limit: float = 0.0, alpha: float = 1.0, n_tiles=None, tile_rows: int = 0) -> torch.Tensor:
-    """[rows, 2F] = [gate | up] -> [rows, F]; ACT_RELU2: [rows, F] -> relu(.)^2 of it, no up half.  See kb2_seq_glu for the kinds."""
+def glu(gate_up: torch.Tensor, out_dtype, kind: int, limit: float = 0.0, alpha: float = 1.0, n_tiles=None, tile_rows: int = 0, bias=None,
+        row_w=None, row_map=None) -> torch.Tensor:
+    """[rows, 2F] = [gate | up] -> [rows, F]; ACT_RELU2: [rows, F] -> relu(.)^2 of it, no up half.  See kb2_seq_glu for the kinds.
+    bias [2F] fp32 joins the two halves.  row_w fp32: both halves of row r are first multiplied by row_w[r] (row_w[row_map[r]] with an
+    int32 row_map, 0 for a negative entry) — a weight on the input of the unit."""
     rows, F2 = gate_up.shape
     F = F2 if kind == ACT_RELU2 else F2 // 2
     out = torch.empty((rows, F), dtype=out_dtype, device=gate_up.device)
     check(load().kb2_seq_glu(gate_up.data_ptr(), dt_code(gate_up.dtype), gate_up.stride(0), out.data_ptr(), dt_code(out_dtype), rows, F,
-                             int(kind), float(limit), float(alpha), _ptr(n_tiles), int(tile_rows), _s(gate_up)))
+                             int(kind), float(limit), float(alpha), _ptr(n_tiles), int(tile_rows), _ptr(bias), _ptr(row_w), _ptr(row_map),
+                             _s(gate_up)))
     return out
 
 
@@ -278,13 +286,31 @@ def residual_scale_rms(x, y=None, y_mult: float = 1.0, norm=None, w_shift: float
     return h
 
 
-def conv(proj: torch.Tensor, C: int, taps: torch.Tensor, bias, act: bool, tail: torch.Tensor, tb: "StepTables", bias_after: bool = False) -> torch.Tensor:
+def residual_post_rms(x, y=None, norm=None, mult: float = 1.0, y2=None, coefs=(1.0, 1.0), bias=None, out_norm=None, out_dtype=None, eps=1e-5):
+    """Norm on the sublayer's output only.  z = coefs[0] y + coefs[1] y2 + bias; x (fp32, in place) += mult * z / rms(z) * norm.  Returns x in
+    out_dtype — x itself for float32 — or, with out_norm, x / rms(x) * out_norm in a buffer of its own; None without out_dtype."""
+    T, W = x.shape
+    for t in (x, y, y2):
+        if t is not None and (t.dtype != torch.float32 or not t.is_contiguous() or t.shape != x.shape):
+            raise ValueError("residual_post_rms: x and the addends must be contiguous fp32 of one shape")
+    for t in (norm, bias, out_norm):
+        if t is not None and (t.dtype != torch.float32 or t.numel() != W):
+            raise ValueError("residual_post_rms: weights and bias are fp32 of x's width")
+    h = None
+    if out_dtype is not None and (out_norm is not None or out_dtype != torch.float32):
+        h = torch.empty((T, W), dtype=out_dtype, device=x.device)
+    if y is not None or h is not None:
+        check(load().kb2_seq_residual_post_rms(x.data_ptr(), _ptr(y), float(coefs[0]), _ptr(y2), float(coefs[1]), _ptr(bias), float(mult), _ptr(norm),
+                                               _ptr(out_norm), _ptr(h), dt_code(h.dtype) if h is not None else 0, T, W, float(eps), _s(x)))
+    return x if h is None and out_dtype is not None else h
+
+
+def conv(proj: torch.Tensor, C: int, taps: torch.Tensor, bias, act: bool, tail: torch.Tensor, tb: "StepTables", bias_out=None) -> torch.Tensor:
     """Short causal convolution over time on the first C columns of proj [T, >= C] fp32 (+ bias), with the carried tail
-    [slots, C, taps - 1] read and advanced; silu on the result if act.  bias_after: the bias is added to the convolution's result
-    (ahead of the activation) instead of to its inputs."""
+    [slots, C, taps - 1] read and advanced; bias_out is added to the result, then silu if act."""
     T, K = proj.shape[0], taps.shape[1]
     out = torch.empty((T, C), dtype=torch.float32, device=proj.device)
-    check(load().kb2_seq_conv(proj.data_ptr(), proj.stride(0), T, tb.S, C, K, taps.data_ptr(), _ptr(bias), int(bool(act)) + 2 * int(bool(bias_after)), tail.data_ptr(),
+    check(load().kb2_seq_conv(proj.data_ptr(), proj.stride(0), T, tb.S, C, K, taps.data_ptr(), _ptr(bias), _ptr(bias_out), int(bool(act)), tail.data_ptr(),
                               tb.seq_of.data_ptr(), tb.cu.data_ptr(), tb.slots.data_ptr(), out.data_ptr(), _s(proj)))
     return out
 
@@ -319,12 +345,19 @@ def rms_rows(x: torch.Tensor, w: torch.Tensor, eps: float, out_dtype) -> torch.T
     return out
 
 
-def head_norm_gate(o: torch.Tensor, H: int, dv: int, out_dtype, norm=None, eps: float = 0.0, gate=None, gate_act: str = "silu") -> torch.Tensor:
-    """o [T, >= H dv] fp32 -> per head o / rms(o) * norm (if norm) times silu | sigmoid of gate [T, >= H dv] (if gate), in out_dtype."""
+def head_norm_gate(o: torch.Tensor, H: int, dv: int, out_dtype, norm=None, eps: float = 0.0, gate=None, gate_act: str = "silu",
+                   den=None) -> torch.Tensor:
+    """o [T, >= H dv] fp32 -> per head o / rms(o) * norm (if norm) times silu | sigmoid of gate [T, >= H dv] (if gate), in out_dtype.
+    norm [dv] is shared by the heads, [H dv] has weights of its own for every head.  den [T, H]: o is divided by it first."""
     T = o.shape[0]
+    if norm is not None and norm.numel() not in (dv, H * dv):
+        raise ValueError("head_norm_gate: norm weights per head or shared")
+    if den is not None and (den.dtype != torch.float32 or not den.is_contiguous() or den.numel() != T * H):
+        raise ValueError("head_norm_gate: den [T, H] fp32")
     out = torch.empty((T, H * dv), dtype=out_dtype, device=o.device)
     check(load().kb2_seq_head_norm_gate(o.data_ptr(), o.stride(0), _ptr(norm), float(eps), _ptr(gate), gate.stride(0) if gate is not None else 0,
-                                        {"silu": 0, "sigmoid": 1}[gate_act], T, H, dv, out.data_ptr(), dt_code(out_dtype), _s(o)))
+                                        {"silu": 0, "sigmoid": 1}[gate_act], T, H, dv, out.data_ptr(), dt_code(out_dtype), _ptr(den),
+                                        int(norm is not None and norm.numel() != dv), _s(o)))
     return out
 
 
