@@ -486,7 +486,7 @@ def main():
     ap.add_argument("--cpu-format", default="int4", choices=["int4", "gguf"],
                     help="CPU arm: int4 = moe_forward_unified on INT4 g128 (default); gguf = moe_forward_gguf on native Q4_K/Q8_0 blocks "
                          "(BASELINE configs[0]: --config v2lite --impl reference --cpu-format gguf --tokens 2048)")
-    ap.add_argument("--arch", default="moe", choices=["moe", "vofelix", "megolorn", "gurozen", "zaronex", "kugalorn"],
+    ap.add_argument("--arch", default="moe", choices=["moe", "vofelix", "megolorn", "gurozen", "zaronex", "kugalorn", "kivurax"],
                     help="moe (default): the BASELINE workload above; vofelix: prefill / decode throughput of the ragged-batch model at "
                          "real layer sizes beside the Gated-DeltaNet and MLA blocks at equal size (1 GPU); megolorn: the same for the "
                          "differential-attention / routed-expert model beside Vofelix and the GQA block at equal size; gurozen: the same for "
@@ -494,7 +494,9 @@ def main():
                          "zaronex: the same for the depth-averaged model of side-by-side mixers (pooled-block attention, gated linear "
                          "attention, selective scan, latent attention) beside the Gurozen and Vofelix blocks, with its new kernels alone; "
                          "kugalorn: the same for the model of several mixed stream copies (attention with a distance penalty, latent "
-                         "attention, clamped-swish experts) beside the Zaronex, Gurozen, Megolorn and Vofelix blocks and kernels")
+                         "attention, clamped-swish experts) beside the Zaronex, Gurozen, Megolorn and Vofelix blocks and kernels; "
+                         "kivurax: the same for the model of matrix memory, gated recurrent blocks beside attention, delta rule and experts "
+                         "weighted on their inputs, beside the Zaronex, Megolorn and Gurozen blocks and kernels")
     args = ap.parse_args()
     if args.arch == "vofelix":
         from krasis_b200.bench_seq import run as run_seq
@@ -515,6 +517,10 @@ def main():
     if args.arch == "kugalorn":
         from krasis_b200.bench_seq import run_kugalorn
         run_kugalorn(args, peaks())
+        return
+    if args.arch == "kivurax":
+        from krasis_b200.bench_seq import run_kivurax
+        run_kivurax(args, peaks())
         return
     args.tokens = args.tokens or DEFAULT_TOKENS[args.config]
     if args.impl == "reference":

@@ -1,4 +1,4 @@
-"""Throughput of the ragged-batch models (Vofelix, Megolorn, Gurozen, Zaronex, Kugalorn) at layer sizes of real models, beside the framework's closest existing blocks at
+"""Throughput of the ragged-batch models (Vofelix, Megolorn, Gurozen, Zaronex, Kugalorn, Kivurax) at layer sizes of real models, beside the framework's closest existing blocks at
 equal size: prefill tokens/s (one prompt, whole and in portions), decode tokens/s (several live requests, one token each per step),
 and per-mixer times — the gated delta mixer against the Gated-DeltaNet block, windowed latent attention against the MLA block.
 Random weights; device timing with CUDA events after warm-up; the weights of a step exceed the L2 cache."""
@@ -776,6 +776,167 @@ def run_kugalorn(args, peaks):
     by = 4 * (ctx + 1) * 576 * 2
     kernel("latent_attn_gate_per_head_decode_4", lambda: decode_latent(ql4[:, Hl * 192 + 576:].data_ptr()), by)
     kernel("latent_attn_decode_4 (like kernel: Vofelix)", lambda: decode_latent(None), by)
+    out["blocks_at_equal_size"] = blk
+    out["kernels"] = kern
+    out["peaks"] = peaks
+    print(json.dumps(out))
+
+
+def kivurax_config(width=2048, vocab=32768, window=1024, experts=64, top=6, expert_ff=1024):
+    """Matrix memory with the state size of Zaronex's gated linear attention (32 heads, 128 x 128), the delta rule at Vofelix's geometry, windowed
+    attention at Zaronex's (16 heads x 128 over 2 key/value heads) beside a recurrent block as wide as Zaronex's selective scan (4096 channels,
+    gates in 16 blocks of 256), Megolorn's number and size of experts, dense units of four times the width."""
+    memory = {"heads": 32, "dim": 128, "vdim": 128, "gate_cap": 15.0}
+    delta = {"heads": 32, "kv_heads": 16, "dim": 128, "vdim": 128, "conv": 4}
+    left = {"heads": 16, "kv_heads": 2, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": window},
+            "rot": {"base": 1000000.0, "dims": 128, "scaling": {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+    right = {"width": 2 * width, "blocks": 16, "conv": 4}
+    par = {"left": left, "right": right, "left_scale": 0.7, "right_scale": 0.7}
+    dense = {"kind": "dense", "ff": 4 * width}
+    moe = {"kind": "moe", "router": {"experts": experts, "top": top}, "expert": {"ff": expert_ff}}
+    layers = [{"type": t, "mixer": m, "mlp": f} for t, m, f in (("mlstm", memory, dense), ("parallel", par, moe), ("delta", delta, moe), ("mlstm", memory, dense))]
+    return {"architecture": "Kivurax", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "residual_mult": 0.5, "layers": layers}
+
+
+def run_kivurax(args, peaks):
+    from . import capi, seqops as ops
+    from .build import build, build_seq
+    build_seq()
+    build()                                          # the tcgen05 GEMM and attention core serve long bfloat16 steps
+    from .attention import RecurrentStatePool
+    from .kivurax import KivuraxConfig, KivuraxModel
+    dev = torch.device("cuda", 0)
+    tokens = args.tokens or 4096
+    cfg = KivuraxConfig.from_dict(kivurax_config())
+    model = KivuraxModel.random(cfg, seed=0, dtype=torch.bfloat16, device=0)
+    g = torch.Generator().manual_seed(0)
+    prompt = torch.randint(0, cfg.vocab, (tokens,), generator=g).tolist()
+    out = {"metric": "kivurax_prefill_tokens_per_s", "unit": "tokens/s", "n_gpus": 1, "steps": args.steps, "warmup": args.warmup,
+           "higher_is_better": True, "dtype": "bf16", "data": "synthetic (random weights and token ids)", "vs_baseline": None,
+           "config": {"model": "kivurax width 2048: 4 layers (matrix memory 32 heads 128 x 128 | attention 16 heads x 128 / 2 kv heads, window 1024, "
+                               "beside a recurrent block of 4096 channels | delta rule 32 / 16 heads x 128 | matrix memory); dense ff 8192 in the "
+                               "outer layers, 64 experts, top 6, expert ff 1024 in the inner ones", "prompt_tokens": tokens,
+                      "l2": "weights of one step (about 2.1 GB) exceed L2"}}
+    _serving(model, args, prompt, out)
+
+    # ---- per-block times, prefill and decode, beside the closest blocks of the other designs at equal size
+    blk, W, ctx = {}, cfg.width, 2048
+    h = (torch.randn(tokens, W, generator=g) * 0.5).to(torch.bfloat16).to(dev)
+    h4 = h[:4].contiguous()
+    tb = ops.StepTables([(prompt, 0, 0, list(range((tokens + 63) // 64)))], dev)
+    tb4 = ops.StepTables([([1], ctx, r, list(range(r * 40, r * 40 + 33))) for r in range(4)], dev)
+    model.make_caches(max(tokens, 4 * 40 * 64) + 64, 4)
+    kc, vc = model.kv_cache.get_layer_caches(0)
+    for t in (kc, vc):                               # finite, ordinary contents: what decode reads at once
+        t.copy_((torch.randn(t.shape, device=dev) * 0.5).to(t.dtype))
+    memory, pair, delta = (model.layers[i]["mixer"] for i in range(3))
+    dense, moe = model.layers[0]["mlp"], model.layers[1]["mlp"]
+    st = model._state
+
+    def both(name, fn_of):                           # fn_of(h, tables) -> callable
+        blk[name + "_ms"] = round(_time(fn_of(h, tb), 2, 5), 3)
+        blk["decode_4_tokens_" + name + "_ms"] = round(_time(fn_of(h4, tb4), 3, 20), 4)
+    both("matrix_memory_mixer", lambda hh, t: (lambda: memory.forward(hh, t, *st[0])))
+    both("keys_as_values_attention_block", lambda hh, t: (lambda: pair.left.forward(hh, t, kc, vc, 64)))
+    both("recurrent_block", lambda hh, t: (lambda: pair.right.forward(hh, t, *st[1])))
+    both("delta_mixer", lambda hh, t: (lambda: delta.forward(hh, t, *st[2])))
+    both("dense_ff_8192_with_biases", lambda hh, t: (lambda: dense.forward(hh)))
+    both("routed_experts_block", lambda hh, t: (lambda: moe.forward(hh)))
+    zm = None
+    try:                                             # the closest blocks of the other designs, built at this design's sizes
+        from .megolorn import MegolornConfig, MegolornModel
+        from .zaronex import ZaronexConfig, ZaronexModel
+        zraw = zaronex_config()
+        zraw["layers"] = [dict(zraw["layers"][1]), dict(zraw["layers"][2], mlp=None)]
+        zm = ZaronexModel.random(ZaronexConfig.from_dict(zraw), seed=0, dtype=torch.bfloat16, device=0)
+        pool = RecurrentStatePool(4, dev)
+        gla, scan, za = zm.layers[0]["mixer"].right, zm.layers[1]["mixer"].right, zm.layers[1]["mixer"].left
+        gst, sst = gla.register_state(pool), scan.register_state(pool)
+        both("zaronex_gated_linear_attention_mixer", lambda hh, t: (lambda: gla.forward(hh, t, gst)))
+        both("zaronex_selective_scan_mixer", lambda hh, t: (lambda: scan.forward(hh, t, *sst)))
+        both("zaronex_rotated_value_attention_block", lambda hh, t: (lambda: za.forward(hh, t, kc, vc, 64)))
+        both("zaronex_dense_ff_8192", lambda hh, t: (lambda: zm.layers[0]["mlp"].forward(hh)))
+        mraw = megolorn_config(experts=64, identity=0)
+        mraw["layers"] = [dict(mraw["layers"][0], mlp={k: v for k, v in mraw["layers"][1]["mlp"].items() if k != "shared"})]
+        mm = MegolornModel.random(MegolornConfig.from_dict(mraw), seed=0, dtype=torch.bfloat16, device=0)
+        both("megolorn_routed_experts_block", lambda hh, t: (lambda: mm.layers[0]["mlp"].forward(hh)))
+    except Exception as exc:       # noqa: BLE001 — the comparison is optional; the new design's numbers stand without it
+        blk["comparison_unavailable"] = f"{type(exc).__name__}: {exc}"
+
+    # ---- the new kernels alone, each beside the like kernel: time, algorithmic bytes and flops, fractions of the measured peaks
+    kern, lib, core = {}, ops.load(), capi.load()
+    cs = torch.cuda.current_stream(dev).cuda_stream
+    fma_tflops = 148 * 128 * 2 * 1.965e9 / 1e12      # fp32 FMA lanes x 2 flops x max SM clock: the ceiling of a recurrence on CUDA cores
+
+    def kernel(name, fn, nbytes, flops=0.0, reps=(3, 10)):
+        ms_k = _time(fn, *reps)
+        e = {"ms": round(ms_k, 4), "GB_per_s": round(nbytes / ms_k / 1e6, 1), "of_measured_hbm": round(nbytes / ms_k / 1e6 / peaks["hbm_gbs"], 3)}
+        if flops:
+            e.update(TFLOP_per_s=round(flops / ms_k / 1e9, 2), of_fp32_fma_ceiling=round(flops / ms_k / 1e9 / fma_tflops, 3))
+        kern[name] = e
+    rnd = lambda *s: torch.randn(*s, device=dev)
+    H, dk, dv, C, B = memory.H, memory.dk, memory.dv, pair.right.C, pair.right.B
+    for label, T_, t in (("prefill_4096", tokens, tb), ("decode_4", 4, tb4)):
+        S_ = t.S
+        proj, o, small = rnd(T_, memory.w_in.shape[0]) * 0.3, torch.empty(T_, H * dv, device=dev), torch.empty(4, T_, H, device=dev)
+        s0, n0, m0 = st[0]
+        kernel(f"matrix_memory_{label}", lambda: ops.check(lib.kb2_seq_mlstm(
+            proj.data_ptr(), proj.stride(0), memory.q_off, memory.k_off, memory.v_off, memory.i_off, memory.f_off, memory.i_b.data_ptr(),
+            memory.f_b.data_ptr(), memory.cap, dk ** -0.5, T_, S_, H, dk, dv, s0.data_ptr(), n0.data_ptr(), m0.data_ptr(), t.cu.data_ptr(),
+            t.slots.data_ptr(), small.data_ptr(), o.data_ptr(), small[3].data_ptr(), cs)),
+               T_ * (2 * H * dk + 2 * H * dv + 3 * H) * 4 + 2 * S_ * H * dk * (dv + 1) * 4, flops=4.0 * T_ * H * dk * dv)
+        dec, gsc, gs_ = rnd(T_, H * dk), torch.empty(T_, H * dk, device=dev), torch.zeros(4, H, dk, dv, device=dev)
+        qkv = rnd(T_, 2 * H * dk + 2 * H * dv) * 0.3
+        kernel(f"gla_scan_{label} (like kernel: Zaronex)", lambda: ops.check(lib.kb2_seq_gla(
+            qkv.data_ptr(), qkv.stride(0), 0, H * dk, 2 * H * dk, dec.data_ptr(), H * dk, None, 16.0, dk ** -0.5, T_, S_, H, dk, dv, gs_.data_ptr(),
+            t.cu.data_ptr(), t.slots.data_ptr(), gsc.data_ptr(), o.data_ptr(), cs)),
+               T_ * (3 * H * dk + 2 * H * dv) * 4 + 2 * S_ * H * dk * dv * 4, flops=4.0 * T_ * H * dk * dv)
+        og, den = torch.empty(T_, H * dv, dtype=torch.bfloat16, device=dev), rnd(T_, H).abs() + 1
+        kernel(f"head_norm_divisor_gate_{label}", lambda: ops.head_norm_gate(o, H, dv, torch.bfloat16, norm=memory.norm, eps=1e-5, gate=qkv[:, :H * dv],
+                                                                              gate_act="sigmoid", den=den), T_ * H * dv * 10)
+        nw = torch.ones(dv, device=dev)
+        kernel(f"head_norm_gate_{label} (like kernel: Zaronex)",
+               lambda: ops.head_norm_gate(o, H, dv, torch.bfloat16, norm=nw, eps=1e-5, gate=qkv[:, :H * dv], gate_act="silu"), T_ * H * dv * 10)
+        del og
+        u, z, p2 = rnd(T_, C), rnd(T_, 2 * C), rnd(T_, 2 * C)
+        y = torch.empty(T_, C, dtype=torch.bfloat16, device=dev)
+        ru = pair.right
+        kernel(f"rglru_scan_{label}", lambda: ops.check(lib.kb2_seq_rglru(
+            u.data_ptr(), C, z.data_ptr(), 2 * C, 2 * ru.bs, p2[:, C:].data_ptr(), 2 * C, ru.ra_b.data_ptr(), ru.ri_b.data_ptr(), ru.y_b.data_ptr(),
+            ru.lam.data_ptr(), T_, S_, C, ru.bs, st[1][1].data_ptr(), t.cu.data_ptr(), t.slots.data_ptr(), y.data_ptr(), 1, cs)),
+               T_ * C * (16 + 2) + 2 * S_ * C * 4)
+        kernel(f"recurrent_block_gate_products_{label}", lambda: ru._gate_products(u), T_ * C * 12 + 2 * C * ru.bs * 2,
+               flops=4.0 * T_ * C * ru.bs)
+        if zm is not None:
+            xp, sst2 = rnd(T_, scan.R + 2 * scan.N), torch.zeros(4, C, scan.N, device=dev)
+            kernel(f"selective_scan_{label} (like kernel: Zaronex)", lambda: ops.check(lib.kb2_seq_selective_scan(
+                u.data_ptr(), C, z.data_ptr(), 2 * C, scan.dt_b.data_ptr(), xp.data_ptr(), scan.R + 2 * scan.N, scan.R, p2.data_ptr(), 2 * C, C,
+                scan.A_log.data_ptr(), scan.D.data_ptr(), T_, S_, C, scan.N, sst2.data_ptr(), t.cu.data_ptr(), t.slots.data_ptr(), y.data_ptr(), 1, cs)),
+                   T_ * (3 * C * 4 + C * 2 + 2 * scan.N * 4) + 2 * S_ * C * scan.N * 4 + C * scan.N * 4, flops=6.0 * T_ * C * scan.N)
+        conv_args = (p2, C, ru.taps)
+        tail = st[1][0]
+        kernel(f"conv_two_biases_{label}", lambda: ops.conv(*conv_args, ru.x_b, False, tail, t, bias_out=ru.conv_b), T_ * C * 8)
+        kernel(f"conv_silu_{label} (like kernel: Vofelix)", lambda: ops.conv(*conv_args, None, True, tail, t), T_ * C * 8)
+        x, ya, yb, w = rnd(T_, W), rnd(T_, W), rnd(T_, W), rnd(W)
+        kernel(f"residual_post_rms_{label}", lambda: ops.residual_post_rms(x, ya, w, 0.5, bias=w, out_dtype=torch.bfloat16), T_ * W * 14)
+        kernel(f"residual_post_rms_two_terms_{label}", lambda: ops.residual_post_rms(x, ya, w, 0.5, y2=yb, coefs=(0.7, 0.7), out_dtype=torch.bfloat16), T_ * W * 18)
+        kernel(f"residual_scale_rms_{label} (like kernel: Gurozen)", lambda: ops.residual_scale_rms(x, ya, 0.5, norm=w, out_dtype=torch.bfloat16), T_ * W * 14)
+        gu = (rnd(T_, 2 * 4 * W)).to(torch.bfloat16)
+        fb, rw = rnd(2 * 4 * W), rnd(T_)
+        by = T_ * 4 * W * 6
+        kernel(f"glu_bias_{label}", lambda: ops.glu(gu, torch.bfloat16, ops.GLU_SILU, bias=fb), by)
+        kernel(f"glu_row_weight_{label}", lambda: ops.glu(gu, torch.bfloat16, ops.GLU_SILU, row_w=rw), by)
+        kernel(f"glu_{label} (like kernel: Megolorn)", lambda: ops.glu(gu, torch.bfloat16, ops.GLU_SILU), by)
+    att = pair.left
+    Hq, G, d, win = att.H, att.G, att.d, att.window
+    q, k, v = (rnd(tokens, n * d).to(torch.bfloat16) for n in (Hq, G, G))
+    o = torch.empty(tokens, Hq * d, device=dev)
+    pairs = sum(min(i + 1, win) for i in range(tokens))
+    core_args = (q.data_ptr(), k.data_ptr(), v.data_ptr(), o.data_ptr(), tokens, 0, tokens, Hq, G, 1, d, d ** -0.5, 0.0, win)
+    for name, sink in (("attention_core_one_added_prefill_4096", att.sink), ("attention_core_prefill_4096 (like kernel: Zaronex, no sink)", None)):
+        kernel(name, lambda: capi.check(core.kb2_fmha_maps_sink(*core_args, ops._ptr(sink), None, 0, cs)), tokens * (Hq * d * 6 + 4 * G * d), 4.0 * pairs * Hq * d)
+        kern[name]["of_measured_bf16"] = round(kern[name]["TFLOP_per_s"] / peaks["tf_burst"], 3)
+        del kern[name]["of_fp32_fma_ceiling"]
     out["blocks_at_equal_size"] = blk
     out["kernels"] = kern
     out["peaks"] = peaks
