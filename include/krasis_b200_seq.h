@@ -230,10 +230,10 @@ KB2SEQ_API int kb2_seq_mlstm(const float* proj, long long ld, int q_off, int k_o
 
 /* Real-gated linear recurrent unit over each sequence's portion, C channels in blocks of bs.  u [T, ldu]: inputs; z: gate products, the
  * pair of channel c = b bs + j of token t at z[t ldz + b zb + j] (recurrence gate r) and z[t ldz + b zb + bs + j] (input gate i);
- * y [T, ldy]: the other branch; biases [C] may be null.  log a = -8 sigmoid(r) softplus(lam), S <- a S + sqrt(1 - a^2) sigmoid(i) u,
+ * y [T, ldy]: the other branch; biases [C] may be null.  log a = rate sigmoid(r) with rate [C] <= 0 (-8 softplus(lam) in Griffin), S <- a S + sqrt(1 - a^2) sigmoid(i) u,
  * out [T, C] = S gelu_tanh(y) in dt_out; state [slots][C] fp32 is read and written back. */
 KB2SEQ_API int kb2_seq_rglru(const float* u, long long ldu, const float* z, long long ldz, long long zb, const float* y, long long ldy,
-                             const float* r_bias, const float* i_bias, const float* y_bias, const float* lam, int T, int S, int C, int bs,
+                             const float* r_bias, const float* i_bias, const float* y_bias, const float* rate, int T, int S, int C, int bs,
                              float* state, const int* cu, const int* slots, void* out, int dt_out, void* stream);
 
 /* out [blocks][T_pad][2 bs] bf16: row (b, t) = [high | low] parts of u[t, b bs .. b bs + bs), whose sum is the fp32 value to 2^-17 of its

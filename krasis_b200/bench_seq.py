@@ -903,7 +903,7 @@ def run_kivurax(args, peaks):
         ru = pair.right
         kernel(f"rglru_scan_{label}", lambda: ops.check(lib.kb2_seq_rglru(
             u.data_ptr(), C, z.data_ptr(), 2 * C, 2 * ru.bs, p2[:, C:].data_ptr(), 2 * C, ru.ra_b.data_ptr(), ru.ri_b.data_ptr(), ru.y_b.data_ptr(),
-            ru.lam.data_ptr(), T_, S_, C, ru.bs, st[1][1].data_ptr(), t.cu.data_ptr(), t.slots.data_ptr(), y.data_ptr(), 1, cs)),
+            ru.rate.data_ptr(), T_, S_, C, ru.bs, st[1][1].data_ptr(), t.cu.data_ptr(), t.slots.data_ptr(), y.data_ptr(), 1, cs)),
                T_ * C * (16 + 2) + 2 * S_ * C * 4)
         kernel(f"recurrent_block_gate_products_{label}", lambda: ru._gate_products(u), T_ * C * 12 + 2 * C * ru.bs * 2,
                flops=4.0 * T_ * C * ru.bs)

@@ -7,8 +7,8 @@ Two targets, so that a model only compiles what it runs on:
                                   key channel) with state slots, per-head paged multi-map attention (score cap, sink, pooled blocks
                                   before the window, rotated values, distance penalty), gated and ungated linear units, router and
                                   routed experts,
-                                  gated linear attention and selective scan with state slots, side-by-side mixers, depth average,
-                                  several mixed copies of the residual stream
+                                  gated linear attention, matrix memory (mLSTM), selective scan and real-gated linear recurrent unit with
+                                  state slots, side-by-side mixers, depth average, several mixed copies of the residual stream
 nvcc cross-compiles without a GPU.  The .so files are git-ignored; a missing or stale one is rebuilt on demand.
 """
 import hashlib

@@ -505,10 +505,17 @@ __global__ void glu_bf16x8_kernel(const bf16* __restrict__ in, long long ld_in, 
       }
     }
     if (bias != nullptr) {
+      float ba[8], bb[8] = {};                     // f and F are multiples of 8, the launcher checks the base: 16-byte loads
+      *reinterpret_cast<float4*>(ba) = *reinterpret_cast<const float4*>(bias + f);
+      *reinterpret_cast<float4*>(ba + 4) = *reinterpret_cast<const float4*>(bias + f + 4);
+      if (kind != 3) {
+        *reinterpret_cast<float4*>(bb) = *reinterpret_cast<const float4*>(bias + F + f);
+        *reinterpret_cast<float4*>(bb + 4) = *reinterpret_cast<const float4*>(bias + F + f + 4);
+      }
 #pragma unroll
       for (int e = 0; e < 8; ++e) {
-        a[e] += bias[f + e];
-        if (kind != 3) b[e] += bias[F + f + e];
+        a[e] += ba[e];
+        b[e] += bb[e];
       }
     }
     uint4 o;
@@ -919,7 +926,7 @@ KB2SEQ_API int kb2_seq_glu(const void* in, int dt_in, long long ld_in, void* out
                            void* stream) {
   if (!in || !out || rows <= 0 || F <= 0 || ld_in < (kind == 3 ? F : 2 * F) || kind < 0 || kind > 3 || bad_dt(dt_in) || bad_dt(dt_out))
     return failf(KB2SEQ_ERR_VALUE, "glu: bad argument");
-  if (dt_in == 1 && dt_out == 1 && F % 8 == 0 && ld_in % 8 == 0 && !((uintptr_t)in & 15) && !((uintptr_t)out & 15)) {
+  if (dt_in == 1 && dt_out == 1 && F % 8 == 0 && ld_in % 8 == 0 && !((uintptr_t)in & 15) && !((uintptr_t)out & 15) && !((uintptr_t)bias & 15)) {
     const long long n8 = rows * (F / 8);
     const unsigned blocks8 = (unsigned)((n8 + 255) / 256 > 148 * 16 ? 148 * 16 : (n8 + 255) / 256);
     glu_bf16x8_kernel<<<blocks8, 256, 0, (cudaStream_t)stream>>>((const bf16*)in, ld_in, (bf16*)out, rows, F, kind, limit, alpha, n_tiles, tile_rows, bias, row_w,

@@ -5,8 +5,9 @@
 //                          channel alpha = sigmoid(z)^(1 / tau); the state of a (sequence, head, slice of value columns) lives in
 //                          registers: a generic form (P lanes share a column and each keeps dk / P of its rows) and, for key sizes
 //                          32 / 64 / 128 / 256, a form with lane = column, warp = slice of rows and cp.async token tiles
-//                          the same two kernels serve the matrix memory of mLSTM, S <- keep_t S + add_t k_t v_t^T with one pair of numbers per
-//                          token and head and a further column of ones whose read-out is the normaliser
+//                          the generic form also serves the matrix memory of mLSTM, S <- keep_t S + add_t k_t v_t^T with one pair of numbers
+//                          per token and head and a further column of ones whose read-out is the normaliser
+//   mlstm_reg              the matrix memory for the same key sizes: a lane holds a tile of rows x columns, a warp of its own the key sum
 //   mlstm_gates            log gates of mLSTM and their running maximum m_t = max(f_t + m_(t-1), i_t) by a (sum, maximum) scan; keep and add
 //                          relative to m_t
 //   rglru_scan             real-gated linear recurrent unit: per channel S <- a_t S + sqrt(1 - a_t^2) i_t u_t, times gelu of the other branch;
@@ -306,168 +307,292 @@ __device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
   return r;
 }
 
-// The recurrence of the matrix memory with the layout of gla_reg: a block owns 32 value columns of a (sequence, head), lane = column, warp =
-// DK / 8 rows in registers, two rows per 64-bit register.  One decay per token and head, so k and q are all a token broadcasts; add joins
-// the value.  The last block of a head (blockIdx.z == dv / 32) keeps the key sum: its value is 1 and lane 0 stands for the column.
+// The recurrence of the matrix memory in registers: a block owns 32 value columns of a (sequence, head); warp w keeps DK / 8 rows of them, a
+// lane a tile of R rows x CPL columns (128 keys: 4 x 4), so that a 16-byte read of k, q or v serves several state elements; row pairs sit in
+// 64-bit registers.  Tiles of kMemTile tokens arrive by cp.async, kMemStages deep (the recurrence of a tile is shorter than a trip to memory).
+// The lanes' and warps' pieces of S^T q meet in shared memory while the next tile runs: one barrier per tile.  In the first block of a head
+// (blockIdx.z == 0) one more warp keeps the key sum, DK / 32 rows per lane.
+constexpr int kMemTile = 8, kMemWarps = 8, kMemStages = 4, kMemUnroll = 2;
+static_assert(kMemTile == kMemWarps, "the read-outs take a warp per token of the tile");
+template <int DK> struct MemShape {
+  static constexpr int Q = DK / kMemWarps;             // rows of a warp
+  static constexpr int RG = DK == 32 ? 2 : 4;          // row groups of its lanes; 32 / RG column groups of CPL = RG columns
+  static constexpr int R = Q / RG, CPL = RG;
+  static constexpr int kFloats = kMemStages * kMemTile * (2 * DK + 32 + 4) + 2 * kMemTile * (kMemWarps * RG * 32 + 32 + 1);
+};
+template <int N> __device__ __forceinline__ void ld_vec(const float* p, float* v) {
+  if constexpr (N % 4 == 0) {
+#pragma unroll
+    for (int i = 0; i < N / 4; ++i) {
+      const float4 f = *reinterpret_cast<const float4*>(p + 4 * i);
+      v[4 * i] = f.x; v[4 * i + 1] = f.y; v[4 * i + 2] = f.z; v[4 * i + 3] = f.w;
+    }
+  } else if constexpr (N == 2) {
+    const float2 f = *reinterpret_cast<const float2*>(p);
+    v[0] = f.x; v[1] = f.y;
+  } else {
+    v[0] = p[0];
+  }
+}
+template <int N> __device__ __forceinline__ void st_vec(float* p, const float* v) {
+  if constexpr (N == 4) *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+  else *reinterpret_cast<float2*>(p) = make_float2(v[0], v[1]);
+}
 template <int DK>
-__global__ void __launch_bounds__(32 * kGlaWarps) mlstm_reg_kernel(const float* __restrict__ qkv, long long ld, int q_off, int k_off, int v_off,
+__global__ void __launch_bounds__(32 * (kMemWarps + 1), 1) mlstm_reg_kernel(const float* __restrict__ qkv, long long ld, int q_off, int k_off, int v_off,
                                                                    float q_scale, int H, int dv, float* __restrict__ state,
                                                                    const int* __restrict__ cu, const int* __restrict__ slots,
                                                                    float* __restrict__ out, MemoryGates mg) {
-  constexpr int P = kGlaWarps, NT = 32 * P, Q = DK / P;
+  using M = MemShape<DK>;
+  constexpr int P = kMemWarps, NT = 32 * (P + 1), Q = M::Q, R = M::R, CPL = M::CPL, RG = M::RG, NP = P * RG, KR = DK / 32;
   extern __shared__ __align__(16) float sm[];
-  float* ks = sm;                                   // [2][kGlaTile][DK]
-  float* qs = ks + 2 * kGlaTile * DK;
-  float* vs = qs + 2 * kGlaTile * DK;               // [2][kGlaTile][32]
-  float* gs = vs + 2 * kGlaTile * 32;               // [2][kGlaTile][2]: keep, add
-  float* os_part = gs + 2 * kGlaTile * 2;           // [kGlaTile][P][32]
+  float* ks = sm;                                      // [kMemStages][kMemTile][DK]
+  float* qs = ks + kMemStages * kMemTile * DK;
+  float* vs = qs + kMemStages * kMemTile * DK;         // [kMemStages][kMemTile][32]
+  float* os_part = vs + kMemStages * kMemTile * 32;    // [2][kMemTile][NP][32]
+  float* n_part = os_part + 2 * kMemTile * NP * 32;    // [2][kMemTile][32]
+  float* m_part = n_part + 2 * kMemTile * 32;          // [2][kMemTile]: m of the token
+  float* gs = m_part + 2 * kMemTile;                       // [kMemStages][kMemTile][4]: keep, add, mx, -
   const int s = blockIdx.x, h = blockIdx.y, j0 = blockIdx.z * 32;
-  const bool ones = j0 >= dv;
   const int tid = threadIdx.x, lane = tid & 31, piece = tid >> 5;
+  const int rg = lane / (32 / RG), row0 = piece * Q + rg * R, col0 = (lane % (32 / RG)) * CPL;
   const int t0 = cu[s], n = cu[s + 1] - cu[s];
   const long long head = (long long)slots[s] * H + h;
-  float* Sg = ones ? mg.nstate + head * DK : state + head * DK * dv + j0 + lane;
-  const int pitch = ones ? 1 : dv;
-  uint64_t S[Q / 2];
+  float* Sg = state + head * DK * dv + (long long)row0 * dv + j0 + col0;
+  uint64_t S[R / 2][CPL];                              // S[i][c]: rows row0 + 2 i, row0 + 2 i + 1 of column col0 + c
 #pragma unroll
-  for (int ii = 0; ii < Q / 2; ++ii)
-    S[ii] = pack2(Sg[(long long)(piece * Q + 2 * ii) * pitch], Sg[(long long)(piece * Q + 2 * ii + 1) * pitch]);
+  for (int i = 0; i < R / 2; ++i) {
+    float lo[CPL] = {}, hi[CPL] = {};
+    if (piece < P) {
+      ld_vec<CPL>(Sg + (long long)(2 * i) * dv, lo);
+      ld_vec<CPL>(Sg + (long long)(2 * i + 1) * dv, hi);
+    }
+#pragma unroll
+    for (int c = 0; c < CPL; ++c) S[i][c] = pack2(lo[c], hi[c]);
+  }
+  const bool sums = blockIdx.z == 0 && piece == P;     // the warp of the key sum: rows lane KR .. lane KR + KR - 1
+  float* Ng = mg.nstate + head * DK + lane * KR;
+  float nsum[KR];
+#pragma unroll
+  for (int i = 0; i < KR; ++i) nsum[i] = sums ? Ng[i] : 0.f;
 
   auto load_tile = [&](int buf, int b0) {
-    const int nt = min(kGlaTile, n - b0);
+    const int nt = min(kMemTile, n - b0);
     for (int c = tid; c < nt * (DK / 4); c += NT) {                  // 16-byte chunks of the k and q rows
       const int tt = c / (DK / 4), cc = c - tt * (DK / 4);
-      const long long row = t0 + b0 + tt;
-      const int dst = (buf * kGlaTile + tt) * DK + cc * 4;
-      rec_cp_async16(ks + dst, qkv + row * ld + k_off + h * DK + cc * 4);
-      rec_cp_async16(qs + dst, qkv + row * ld + q_off + h * DK + cc * 4);
+      const float* row = qkv + (long long)(t0 + b0 + tt) * ld + h * DK + cc * 4;
+      const int dst = (buf * kMemTile + tt) * DK + cc * 4;
+      rec_cp_async16(ks + dst, row + k_off);
+      rec_cp_async16(qs + dst, row + q_off);
     }
-    if (!ones)
-      for (int c = tid; c < nt * 8; c += NT) {
-        const int tt = c >> 3, cc = c & 7;
-        rec_cp_async16(vs + (buf * kGlaTile + tt) * 32 + cc * 4, qkv + (long long)(t0 + b0 + tt) * ld + v_off + h * dv + j0 + cc * 4);
-      }
-    if (tid < 2 * nt) rec_cp_async4(gs + buf * kGlaTile * 2 + tid, ((tid & 1) ? mg.add : mg.keep) + (long long)(t0 + b0 + (tid >> 1)) * H + h);
-    rec_cp_async_commit();
+    if (tid < nt * 8) {
+      const int tt = tid >> 3, cc = tid & 7;
+      rec_cp_async16(vs + (buf * kMemTile + tt) * 32 + cc * 4, qkv + (long long)(t0 + b0 + tt) * ld + v_off + h * dv + j0 + cc * 4);
+    }
+    if (tid < 4 * nt && (tid & 3) < 3)
+      rec_cp_async4(gs + buf * kMemTile * 4 + tid, ((tid & 3) == 0 ? mg.keep : (tid & 3) == 1 ? mg.add : mg.mx) + (long long)(t0 + b0 + (tid >> 2)) * H + h);
   };
-
-  load_tile(0, 0);
-  int buf = 0;
-  for (int b0 = 0; b0 < n; b0 += kGlaTile, buf ^= 1) {
-    const int nt = min(kGlaTile, n - b0);
-    rec_cp_async_wait_all();
-    __syncthreads();                                  // tile `buf` is in place; everyone is done with the other buffer and with os_part
-    if (b0 + kGlaTile < n) load_tile(buf ^ 1, b0 + kGlaTile);
-    for (int tt = 0; tt < nt; ++tt) {
-      const int base = (buf * kGlaTile + tt) * DK + piece * Q;
-      const ulonglong2* k4 = reinterpret_cast<const ulonglong2*>(ks + base);
-      const ulonglong2* q4 = reinterpret_cast<const ulonglong2*>(qs + base);
-      const float2 g = *reinterpret_cast<const float2*>(gs + (buf * kGlaTile + tt) * 2);
-      const float vv = (ones ? 1.f : vs[(buf * kGlaTile + tt) * 32 + lane]) * g.y;
-      const uint64_t keep = pack2(g.x, g.x), v2 = pack2(vv, vv);
-      uint64_t a0 = 0, a1 = 0;
 #pragma unroll
-      for (int ii = 0; ii < Q / 4; ++ii) {
-        const ulonglong2 kr = k4[ii], qr = q4[ii];
-        S[2 * ii] = fma2(S[2 * ii], keep, mul2(kr.x, v2));
-        S[2 * ii + 1] = fma2(S[2 * ii + 1], keep, mul2(kr.y, v2));
-        a0 = fma2(S[2 * ii], qr.x, a0);
-        a1 = fma2(S[2 * ii + 1], qr.y, a1);
-      }
-      os_part[(tt * P + piece) * 32 + lane] = sum2(a0) + sum2(a1);
+  for (int st = 0; st < kMemStages - 1; ++st) {
+    if (st * kMemTile < n) load_tile(st, st * kMemTile);
+    rec_cp_async_commit();
+  }
+  // read-out of the tile that starts at b0: a warp per token, a lane per column
+  auto read_out = [&](int b0, int half) {
+    if (piece >= min(kMemTile, n - b0)) return;
+    const long long th = (long long)(t0 + b0 + piece) * H + h;
+    float o0 = 0.f, o1 = 0.f, o2 = 0.f, o3 = 0.f;
+    const float* pp = os_part + (half * kMemTile + piece) * NP * 32 + lane;
+#pragma unroll
+    for (int p = 0; p < NP; p += 4) {
+      o0 += pp[p * 32];
+      o1 += pp[p * 32 + 32];
+      o2 += pp[p * 32 + 64];
+      o3 += pp[p * 32 + 96];
     }
-    __syncthreads();
-    for (int i = tid; i < nt * 32; i += NT) {
-      const int tt = i >> 5, c = i & 31;
-      float o = 0.f;
+    out[th * dv + j0 + lane] = ((o0 + o1) + (o2 + o3)) * q_scale;
+    if (blockIdx.z == 0) {
+      const float nq = warp_sum(n_part[(half * kMemTile + piece) * 32 + lane]);
+      if (lane == 0) mg.den[th] = memory_den(nq * q_scale, m_part[half * kMemTile + piece]);
+    }
+  };
+  int buf = 0, half = 0;
+  for (int b0 = 0; b0 < n; b0 += kMemTile, buf = buf + 1 == kMemStages ? 0 : buf + 1, half ^= 1) {
+    const int nt = min(kMemTile, n - b0), ahead = b0 + (kMemStages - 1) * kMemTile;
+    asm volatile("cp.async.wait_group %0;" ::"n"(kMemStages - 2) : "memory");
+    __syncthreads();                                   // tile `buf` and the pieces of the tile before it are in place; everyone is done with that tile's inputs
+    if (ahead < n) load_tile(buf == 0 ? kMemStages - 1 : buf - 1, ahead);
+    rec_cp_async_commit();                             // a group per tile, empty at the end: the wait above counts groups
+    if (b0 > 0) read_out(b0 - kMemTile, half ^ 1);
+    auto token = [&](int tt, float* o) {
+      const int at = buf * kMemTile + tt;
+      float kf[R], qf[R], v[CPL];
+      ld_vec<R>(ks + at * DK + row0, kf);
+      ld_vec<R>(qs + at * DK + row0, qf);
+      ld_vec<CPL>(vs + at * 32 + col0, v);
+      const float2 g = *reinterpret_cast<const float2*>(gs + at * 4);
+      const uint64_t keep = pack2(g.x, g.x);
+      uint64_t k2[R / 2], q2[R / 2];
 #pragma unroll
-      for (int p = 0; p < P; ++p) o += os_part[(tt * P + p) * 32 + c];
-      const long long th = (long long)(t0 + b0 + tt) * H + h;
-      if (!ones) out[th * dv + j0 + c] = o * q_scale;
-      else if (c == 0) mg.den[th] = memory_den(o * q_scale, mg.mx[th]);
+      for (int i = 0; i < R / 2; ++i) {
+        k2[i] = pack2(kf[2 * i], kf[2 * i + 1]);
+        q2[i] = pack2(qf[2 * i], qf[2 * i + 1]);
+      }
+#pragma unroll
+      for (int c = 0; c < CPL; ++c) {
+        const float va = v[c] * g.y;
+        const uint64_t v2 = pack2(va, va);
+        uint64_t acc = 0;
+#pragma unroll
+        for (int i = 0; i < R / 2; ++i) {
+          S[i][c] = fma2(S[i][c], keep, mul2(k2[i], v2));
+          acc = i == 0 ? mul2(S[i][c], q2[i]) : fma2(S[i][c], q2[i], acc);
+        }
+        o[c] = sum2(acc);
+      }
+    };
+    auto keep_piece = [&](int tt, const float* o) { st_vec<CPL>(os_part + ((half * kMemTile + tt) * NP + piece * RG + rg) * 32 + col0, o); };
+    if (sums) {
+#pragma unroll 2
+      for (int tt = 0; tt < nt; ++tt) {
+        const int at = buf * kMemTile + tt;
+        float kf[KR], qf[KR], o = 0.f;
+        ld_vec<KR>(ks + at * DK + lane * KR, kf);
+        ld_vec<KR>(qs + at * DK + lane * KR, qf);
+        const float2 g = *reinterpret_cast<const float2*>(gs + at * 4);
+#pragma unroll
+        for (int i = 0; i < KR; ++i) {
+          nsum[i] = fmaf(nsum[i], g.x, kf[i] * g.y);
+          o = fmaf(nsum[i], qf[i], o);
+        }
+        n_part[(half * kMemTile + tt) * 32 + lane] = o;
+        if (lane == 0) m_part[half * kMemTile + tt] = gs[at * 4 + 2];
+      }
+    } else if (piece == P) {
+      // nothing to keep in the other blocks
+    } else if (nt == kMemTile) {
+#pragma unroll
+      for (int t4 = 0; t4 < kMemTile; t4 += kMemUnroll) {     // stores after kMemUnroll tokens, so that their loads are in flight together
+        float o[kMemUnroll][CPL];
+#pragma unroll
+        for (int tt = 0; tt < kMemUnroll; ++tt) token(t4 + tt, o[tt]);
+#pragma unroll
+        for (int tt = 0; tt < kMemUnroll; ++tt) keep_piece(t4 + tt, o[tt]);
+      }
+    } else {
+      for (int tt = 0; tt < nt; ++tt) {
+        float o[CPL];
+        token(tt, o);
+        keep_piece(tt, o);
+      }
     }
   }
-  if (ones && lane != 0) return;                       // every lane holds the key sum
+  __syncthreads();
+  if (n > 0) read_out((n - 1) / kMemTile * kMemTile, half ^ 1);
+  if (sums) {
 #pragma unroll
-  for (int ii = 0; ii < Q / 2; ++ii) {
-    float lo, hi;
-    asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(S[ii]));
-    Sg[(long long)(piece * Q + 2 * ii) * pitch] = lo;
-    Sg[(long long)(piece * Q + 2 * ii + 1) * pitch] = hi;
+    for (int i = 0; i < KR; ++i) Ng[i] = nsum[i];
+  }
+  if (piece == P) return;
+#pragma unroll
+  for (int i = 0; i < R / 2; ++i) {
+    float lo[CPL], hi[CPL];
+#pragma unroll
+    for (int c = 0; c < CPL; ++c) asm("mov.b64 {%0, %1}, %2;" : "=f"(lo[c]), "=f"(hi[c]) : "l"(S[i][c]));
+    st_vec<CPL>(Sg + (long long)(2 * i) * dv, lo);
+    st_vec<CPL>(Sg + (long long)(2 * i + 1) * dv, hi);
   }
 }
 
 // ------------------------------------------------------------------------------------------------ real-gated linear recurrent unit
 // u [T, ldu]: convolved inputs of C channels in blocks of bs; z: gate products, the pair of channel c = b bs + j at z + t ldz + b zb + j
 // (recurrence gate) and + bs (input gate); y [T, ldy] the other branch.  Per channel
-//   log a = -8 sigmoid(z_r + r_bias) softplus(lam),  S <- a S + sqrt(1 - a^2) sigmoid(z_i + i_bias) u,  out = S gelu_tanh(y + y_bias).
-// a = 1 + expm1(log a) and 1 - a^2 = -expm1 (2 + expm1): exact where a is next to one.  A block owns 32 channels (lane = channel) of a
-// sequence; warp w takes tokens [4 w, 4 w + 4) of a tile of 4 kRgWarps, composes its (a, b) pairs from S = 0, and the warps' compositions meet
-// in shared memory once per tile.  The next tile's inputs are in registers before this one's are used.
-constexpr int kRgWarps = 16, kRgTok = 4;
-__device__ __forceinline__ float sigmoid_f(float z) { return 1.f / (1.f + expf(-z)); }
-__global__ void __launch_bounds__(32 * kRgWarps) rglru_scan_kernel(const float* __restrict__ u, long long ldu, const float* __restrict__ z,
+//   log a = rate sigmoid(z_r + r_bias),  S <- a S + sqrt(1 - a^2) sigmoid(z_i + i_bias) u,  out = S gelu_tanh(y + y_bias).
+// a = 1 + expm1(log a) and 1 - a^2 = -expm1 (2 + expm1): exact where a is next to one.  A block owns CG groups of 32 channels (lane = channel)
+// of a sequence; warp w of the NW warps of a group takes tokens [TOK w, TOK w + TOK) of a tile, composes its (a, b) pairs from S = 0, and the
+// warps' compositions meet in shared memory once per tile.  The next tile's inputs are in registers before this one's are used.
+// NW = 1 serves steps of single tokens.
+constexpr int kRgWarps = 16, kRgTok = 8, kRgGroups = 4;
+__device__ __forceinline__ float sigmoid_f(float z) { return __fdividef(1.f, 1.f + expf(-z)); }      // both ends come out right: exp = inf gives 0
+__device__ __forceinline__ float sqrt_approx(float x) {
+  float y;
+  asm("sqrt.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+// y gelu's factor: 0.5 (1 + tanh(t)) = sigmoid(2 t)
+__device__ __forceinline__ float gelu_tanh_f(float y) { return y * sigmoid_f(1.5957691216057308f * y * fmaf(0.044715f * y, y, 1.f)); }
+template <int NW, int CG, int TOK>
+__global__ void __launch_bounds__(32 * NW * CG, 1) rglru_scan_kernel(const float* __restrict__ u, long long ldu, const float* __restrict__ z,
                                                                    long long ldz, long long zb, const float* __restrict__ y, long long ldy,
                                                                    const float* __restrict__ r_bias, const float* __restrict__ i_bias,
-                                                                   const float* __restrict__ y_bias, const float* __restrict__ lam, int C, int bs,
+                                                                   const float* __restrict__ y_bias, const float* __restrict__ rate_c, int C, int bs,
                                                                    float* __restrict__ state, const int* __restrict__ cu,
                                                                    const int* __restrict__ slots, void* __restrict__ out, int dt_out) {
-  __shared__ float Aw[2][kRgWarps][32], Bw[2][kRgWarps][32];
-  const int s = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-  const int c = blockIdx.y * 32 + lane;
+  __shared__ float Aw[2][CG][NW][32], Bw[2][CG][NW][32];
+  const int s = blockIdx.x, lane = threadIdx.x & 31, grp = (threadIdx.x >> 5) / NW, warp = (threadIdx.x >> 5) % NW;
+  const int c = (blockIdx.y * CG + grp) * 32 + lane;
   const bool live = c < C;
   const int row0 = cu[s], n = cu[s + 1] - row0;
   float* Sp = state + (long long)slots[s] * C + c;
   float carry = live ? *Sp : 0.f;
   const float rb = live && r_bias ? r_bias[c] : 0.f, ib = live && i_bias ? i_bias[c] : 0.f, yb = live && y_bias ? y_bias[c] : 0.f;
-  const float rate = live ? (float)(-8.0 * softplus_d((double)lam[c])) : 0.f;
+  const float rate = live ? rate_c[c] : 0.f;
   const int blk = live ? c / bs : 0;
-  const float* zc = z + blk * zb + (c - blk * bs);
+  // rows of the next tile's first token of this warp; the tile's tokens lie a row stride apart
+  const long long first = row0 + warp * TOK;
+  const float* zp = z + blk * zb + (c - blk * bs) + first * ldz;
+  const float* up = u + first * ldu + c;
+  const float* yp = y + first * ldy + c;
   struct In { float u, r, i, y; };
-  In cur[kRgTok], nxt[kRgTok];
+  In cur[TOK], nxt[TOK];
   auto load = [&](In* in, int b0) {
 #pragma unroll
-    for (int k = 0; k < kRgTok; ++k) {
-      const int tt = b0 + warp * kRgTok + k;
+    for (int k = 0; k < TOK; ++k) {
+      const int tt = b0 + warp * TOK + k;
       in[k] = {0.f, 0.f, 0.f, 0.f};
-      if (live && tt < n) {
-        const long long t = row0 + tt;
-        in[k] = {u[t * ldu + c], zc[t * ldz], zc[t * ldz + bs], y[t * ldy + c]};
-      }
+      if (live && tt < n) in[k] = {up[k * ldu], zp[k * ldz], zp[k * ldz + bs], yp[k * ldy]};
     }
+    up += NW * TOK * ldu;
+    zp += NW * TOK * ldz;
+    yp += NW * TOK * ldy;
   };
   load(cur, 0);
   int buf = 0;
-  for (int b0 = 0; b0 < n; b0 += kRgWarps * kRgTok, buf ^= 1) {
-    if (b0 + kRgWarps * kRgTok < n) load(nxt, b0 + kRgWarps * kRgTok);
-    float a[kRgTok], b[kRgTok], A = 1.f, B = 0.f;
+  for (int b0 = 0; b0 < n; b0 += NW * TOK, buf ^= 1) {
+    if (b0 + NW * TOK < n) load(nxt, b0 + NW * TOK);
+    float a[TOK], b[TOK], A = 1.f, B = 0.f;
 #pragma unroll
-    for (int k = 0; k < kRgTok; ++k) {
+    for (int k = 0; k < TOK; ++k) {
       a[k] = 1.f;                                     // a place without a token leaves the state as it is
       b[k] = 0.f;
-      if (live && b0 + warp * kRgTok + k < n) {
+      if (live && b0 + warp * TOK + k < n) {
         const float e = expm1f(rate * sigmoid_f(cur[k].r + rb));
         a[k] = 1.f + e;
-        b[k] = sqrtf(-e * (2.f + e)) * sigmoid_f(cur[k].i + ib) * cur[k].u;
+        b[k] = sqrt_approx(-e * (2.f + e)) * sigmoid_f(cur[k].i + ib) * cur[k].u;
       }
       A *= a[k];
       B = fmaf(a[k], B, b[k]);
     }
-    Aw[buf][warp][lane] = A;
-    Bw[buf][warp][lane] = B;
-    __syncthreads();                                  // one barrier per tile: the other buffer is written only after the next one
-    float S = carry, mine = carry;
+    float mine = carry;
+    if constexpr (NW == 1) {
+      carry = fmaf(A, carry, B);
+    } else {
+      Aw[buf][grp][warp][lane] = A;
+      Bw[buf][grp][warp][lane] = B;
+      __syncthreads();                                // one barrier per tile: the other buffer is written only after the next one
+      float S = carry;
 #pragma unroll
-    for (int w = 0; w < kRgWarps; ++w) {
-      if (w == warp) mine = S;
-      S = fmaf(Aw[buf][w][lane], S, Bw[buf][w][lane]);
+      for (int w = 0; w < NW; ++w) {
+        if (w == warp) mine = S;
+        S = fmaf(Aw[buf][grp][w][lane], S, Bw[buf][grp][w][lane]);
+      }
+      carry = S;
     }
-    carry = S;
 #pragma unroll
-    for (int k = 0; k < kRgTok; ++k) {
-      const int tt = b0 + warp * kRgTok + k;
+    for (int k = 0; k < TOK; ++k) {
+      const int tt = b0 + warp * TOK + k;
       mine = fmaf(a[k], mine, b[k]);
-      if (live && tt < n) st_dt(out, dt_out, (long long)(row0 + tt) * C + c, mine * gelu_tanh(cur[k].y + yb));
+      if (live && tt < n) st_dt(out, dt_out, (long long)(row0 + tt) * C + c, mine * gelu_tanh_f(cur[k].y + yb));
       cur[k] = nxt[k];
     }
   }
@@ -641,6 +766,66 @@ __global__ void __launch_bounds__(256) head_norm_gate_kernel(const float* __rest
       v *= gate_act ? 1.f / (1.f + expf(-gz)) : silu(gz);
     }
     st_dt(out, dt_out, wi * dv + j, v);
+  }
+}
+
+// the same for value sizes that are multiples of 4 up to 128 NV and 16-byte rows: a lane keeps its columns in registers
+template <int NV>
+__global__ void __launch_bounds__(256) head_norm_gate_vec_kernel(const float* __restrict__ o, long long ldo, const float* __restrict__ w, float eps,
+                                                                 const float* __restrict__ gate, long long ldg, int gate_act, int H, int dv,
+                                                                 long long T, void* __restrict__ out, int dt_out, const float* __restrict__ den,
+                                                                 int w_heads) {
+  const long long wi = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  const int lane = threadIdx.x & 31;
+  if (wi >= T * H) return;
+  const long long t = wi / H;
+  const int h = (int)(wi - t * H);
+  const float* row = o + t * ldo + (long long)h * dv;
+  const float* gr = gate != nullptr ? gate + t * ldg + (long long)h * dv : nullptr;
+  float4 v[NV], g[NV];
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int j = (lane + 32 * i) * 4;
+    v[i] = j < dv ? *reinterpret_cast<const float4*>(row + j) : make_float4(0.f, 0.f, 0.f, 0.f);
+    if (gr != nullptr && j < dv) g[i] = *reinterpret_cast<const float4*>(gr + j);
+  }
+  const float dinv = den != nullptr ? 1.f / den[wi] : 1.f;
+  float rstd = dinv;
+  if (w != nullptr) {
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const float a = v[i].x * dinv, b = v[i].y * dinv, c = v[i].z * dinv, d = v[i].w * dinv;
+      ss = fmaf(a, a, ss);
+      ss = fmaf(b, b, ss);
+      ss = fmaf(c, c, ss);
+      ss = fmaf(d, d, ss);
+    }
+    rstd = dinv / sqrtf(warp_sum(ss) / (float)dv + eps);
+    if (w_heads) w += (long long)h * dv;
+  }
+  auto act = [&](float z) { return gate_act ? 1.f / (1.f + expf(-z)) : silu(z); };
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int j = (lane + 32 * i) * 4;
+    if (j >= dv) continue;
+    float4 r = make_float4(v[i].x * rstd, v[i].y * rstd, v[i].z * rstd, v[i].w * rstd);
+    if (w != nullptr) {
+      const float4 ww = *reinterpret_cast<const float4*>(w + j);
+      r.x *= ww.x; r.y *= ww.y; r.z *= ww.z; r.w *= ww.w;
+    }
+    if (gr != nullptr) {
+      r.x *= act(g[i].x); r.y *= act(g[i].y); r.z *= act(g[i].z); r.w *= act(g[i].w);
+    }
+    if (dt_out) {
+      const __nv_bfloat162 lo = __floats2bfloat162_rn(r.x, r.y), hi = __floats2bfloat162_rn(r.z, r.w);
+      uint2 p;
+      p.x = *reinterpret_cast<const uint32_t*>(&lo);
+      p.y = *reinterpret_cast<const uint32_t*>(&hi);
+      *reinterpret_cast<uint2*>((bf16*)out + wi * dv + j) = p;
+    } else {
+      *reinterpret_cast<float4*>((float*)out + wi * dv + j) = r;
+    }
   }
 }
 
@@ -845,9 +1030,9 @@ static int launch_gla_scan(const float* qkv, long long ld, int q_off, int k_off,
 template <int DK>
 static int launch_mlstm_reg(const float* qkv, long long ld, int q_off, int k_off, int v_off, float q_scale, int S, int H, int dv, float* state,
                             const int* cu, const int* slots, float* out, const MemoryGates& mg, cudaStream_t st) {
-  const size_t smem = (size_t)(2 * 2 * kGlaTile * DK + 2 * kGlaTile * 34 + kGlaTile * kGlaWarps * 32) * 4;
+  const size_t smem = (size_t)MemShape<DK>::kFloats * 4;
   if (smem > 48 * 1024) SEQ_CUDA(cudaFuncSetAttribute(mlstm_reg_kernel<DK>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-  mlstm_reg_kernel<DK><<<dim3(S, H, dv / 32 + 1), 32 * kGlaWarps, smem, st>>>(qkv, ld, q_off, k_off, v_off, q_scale, H, dv, state, cu, slots, out, mg);
+  mlstm_reg_kernel<DK><<<dim3(S, H, dv / 32), 32 * (kMemWarps + 1), smem, st>>>(qkv, ld, q_off, k_off, v_off, q_scale, H, dv, state, cu, slots, out, mg);
   SEQ_LAUNCHED();
   return KB2SEQ_OK;
 }
@@ -907,8 +1092,9 @@ KB2SEQ_API int kb2_seq_mlstm(const float* proj, long long ld, int q_off, int k_o
   mlstm_gates_kernel<<<dim3(S, H), threads, 0, st>>>(proj, ld, i_off, f_off, i_bias, f_bias, cap, H, mstate, cu, slots, keep, add, mx);
   SEQ_LAUNCHED();
   const MemoryGates mg{keep, add, mx, nstate, den};
-  const bool aligned = ((uintptr_t)proj & 15) == 0 && (ld & 3) == 0 && (q_off & 3) == 0 && (k_off & 3) == 0 && (v_off & 3) == 0;
-  if (aligned && (dk == 32 || dk == 64 || dk == 128 || dk == 256) && dv % 32 == 0 && dv / 32 < 65535) {
+  const bool aligned = (((uintptr_t)proj | (uintptr_t)state) & 15) == 0 && (ld & 3) == 0 && (q_off & 3) == 0 && (k_off & 3) == 0 &&
+                       (v_off & 3) == 0;
+  if (aligned && (dk == 32 || dk == 64 || dk == 128 || dk == 256) && dv % 32 == 0 && dv / 32 <= 65535) {
 #define KB2_MEM(DKV) launch_mlstm_reg<DKV>(proj, ld, q_off, k_off, v_off, q_scale, S, H, dv, state, cu, slots, out, mg, st)
     if (dk == 32) return KB2_MEM(32);
     if (dk == 64) return KB2_MEM(64);
@@ -920,13 +1106,18 @@ KB2SEQ_API int kb2_seq_mlstm(const float* proj, long long ld, int q_off, int k_o
 }
 
 KB2SEQ_API int kb2_seq_rglru(const float* u, long long ldu, const float* z, long long ldz, long long zb, const float* y, long long ldy,
-                             const float* r_bias, const float* i_bias, const float* y_bias, const float* lam, int T, int S, int C, int bs,
+                             const float* r_bias, const float* i_bias, const float* y_bias, const float* rate, int T, int S, int C, int bs,
                              float* state, const int* cu, const int* slots, void* out, int dt_out, void* stream) {
-  if (!u || !z || !y || !lam || !state || !cu || !slots || !out || T <= 0 || S <= 0 || C <= 0 || bs <= 0 || C % bs || bad_dt(dt_out))
+  if (!u || !z || !y || !rate || !state || !cu || !slots || !out || T <= 0 || S <= 0 || C <= 0 || bs <= 0 || C % bs || bad_dt(dt_out))
     return failf(KB2SEQ_ERR_VALUE, "rglru: bad argument");
   if ((C + 31) / 32 > 65535) return failf(KB2SEQ_ERR_VALUE, "rglru: too many channels");
-  rglru_scan_kernel<<<dim3(S, (C + 31) / 32), 32 * kRgWarps, 0, (cudaStream_t)stream>>>(u, ldu, z, ldz, zb, y, ldy, r_bias, i_bias, y_bias, lam, C, bs,
-                                                                                       state, cu, slots, out, dt_out);
+  const int groups = (C + 31) / 32;
+  if (T - S + 1 <= 2)                                  // no portion is longer than two tokens
+    rglru_scan_kernel<1, kRgGroups, 2><<<dim3(S, (groups + kRgGroups - 1) / kRgGroups), 32 * kRgGroups, 0, (cudaStream_t)stream>>>(
+        u, ldu, z, ldz, zb, y, ldy, r_bias, i_bias, y_bias, rate, C, bs, state, cu, slots, out, dt_out);
+  else
+    rglru_scan_kernel<kRgWarps, 1, kRgTok><<<dim3(S, groups), 32 * kRgWarps, 0, (cudaStream_t)stream>>>(
+        u, ldu, z, ldz, zb, y, ldy, r_bias, i_bias, y_bias, rate, C, bs, state, cu, slots, out, dt_out);
   SEQ_LAUNCHED();
   return KB2SEQ_OK;
 }
@@ -968,6 +1159,16 @@ KB2SEQ_API int kb2_seq_head_norm_gate(const float* o, long long ldo, const float
   if (!o || !out || T <= 0 || H <= 0 || dv <= 0 || bad_dt(dt_out) || gate_act < 0 || gate_act > 1)
     return failf(KB2SEQ_ERR_VALUE, "head_norm_gate: bad argument");
   const long long nw = (long long)T * H;
+  const uintptr_t all = (uintptr_t)o | (uintptr_t)w | (uintptr_t)gate | (uintptr_t)out;
+  if (dv % 4 == 0 && dv <= 512 && ldo % 4 == 0 && ldg % 4 == 0 && !(all & 15)) {
+#define KB2_HN(NV)                                                                                                                          \
+  head_norm_gate_vec_kernel<NV><<<(unsigned)((nw + 7) / 8), 256, 0, (cudaStream_t)stream>>>(o, ldo, w, eps, gate, ldg, gate_act, H, dv, T, out, dt_out, \
+                                                                                           den, w_heads)
+    if (dv <= 128) KB2_HN(1); else if (dv <= 256) KB2_HN(2); else KB2_HN(4);
+#undef KB2_HN
+    SEQ_LAUNCHED();
+    return KB2SEQ_OK;
+  }
   head_norm_gate_kernel<<<(unsigned)((nw + 7) / 8), 256, 0, (cudaStream_t)stream>>>(o, ldo, w, eps, gate, ldg, gate_act, H, dv, T, out, dt_out, den,
                                                                                       w_heads);
   SEQ_LAUNCHED();

@@ -409,7 +409,7 @@ class GatedRecurrentUnit:
     """weights: x, y [C, W], x_b, y_b [C], conv [C, taps], conv_b [C], ra, ri [blocks, C / blocks, C / blocks], ra_b, ri_b [blocks, C / blocks],
     lam [C], o [W, C].
 
-    u = conv(x h + x_b) + conv_b; per block r = sigmoid(ra u + ra_b), i = sigmoid(ri u + ri_b); log a = -8 r softplus(lam);
+    u = conv(x h + x_b) + conv_b; per block r = sigmoid(ra u + ra_b), i = sigmoid(ri u + ri_b); log a = -8 r softplus(lam) (`rate` r);
     S <- a S + sqrt(1 - a^2) i u; out = o (S gelu_tanh(y h + y_b)) (the recurrent block of De et al., "Griffin: Mixing Gated Linear
     Recurrences with Local Attention for Efficient Language Models").  The state [slots, C], the convolution's last taps - 1 inputs, the
     gates with their products and the decays are fp32."""
@@ -428,9 +428,10 @@ class GatedRecurrentUnit:
         self.w_in, self.w_o = d(torch.cat(rows, 0)), d(weights["o"])
         opt = lambda k: f(weights[k]).reshape(-1) if k in weights else None
         self.x_b, self.y_b, self.conv_b, self.ra_b, self.ri_b = (opt(k) for k in ("x_b", "y_b", "conv_b", "ra_b", "ri_b"))
-        self.taps, self.lam = f(weights["conv"]), f(weights["lam"])
+        self.taps = f(weights["conv"])
+        self.rate = f(-8.0 * torch.nn.functional.softplus(weights["lam"].double(), threshold=40.0))     # log a at an open recurrence gate
         self.w_gates = d(torch.cat([weights["ra"], weights["ri"]], 1))                        # [blocks, 2 bs, bs]: both gates of a block
-        if self.taps.shape != (self.C, self.K) or self.w_gates.shape != (self.B, 2 * self.bs, self.bs) or self.lam.numel() != self.C:
+        if self.taps.shape != (self.C, self.K) or self.w_gates.shape != (self.B, 2 * self.bs, self.bs) or self.rate.numel() != self.C:
             raise ValueError("recurrent unit: tensor shapes do not match width / blocks / taps")
         # long bfloat16 steps: the gate products of a block run on the tensor cores with the fp32 inputs as a high and a low bfloat16 part
         self.tc_min_tokens = 256
@@ -470,7 +471,7 @@ class GatedRecurrentUnit:
         z, ldz, zb = self._gate_products(u)
         o = torch.empty((T, self.C), dtype=self.dtype, device=h.device)
         ops.check(ops.load().kb2_seq_rglru(u.data_ptr(), u.stride(0), z.data_ptr(), ldz, zb, proj[:, self.C:].data_ptr(), proj.stride(0),
-                                           ops._ptr(self.ra_b), ops._ptr(self.ri_b), ops._ptr(self.y_b), self.lam.data_ptr(), T, tb.S, self.C,
+                                           ops._ptr(self.ra_b), ops._ptr(self.ri_b), ops._ptr(self.y_b), self.rate.data_ptr(), T, tb.S, self.C,
                                            self.bs, state.data_ptr(), tb.cu.data_ptr(), tb.slots.data_ptr(), o.data_ptr(), ops.dt_code(self.dtype),
                                            torch.cuda.current_stream(h.device).cuda_stream))
         return lin(o, self.w_o, torch.float32)
